@@ -18,7 +18,8 @@ reused page are never read: every reader is bounded by the sequence's own length
 
 ``StateNeed`` entries get ``[max_slots, *shape]`` of their dtype each, addressed by slot
 and zeroed when the slot is taken.  Gemma-2 has none; the area exists so that a
-mixer with a recurrent state has a place to keep it.
+mixer with a recurrent state has a place to keep it.  An entry may need both (a mixer that is attention and a
+recurrence side by side); its view is then a :class:`BothView`.
 """
 from __future__ import annotations
 
@@ -70,10 +71,17 @@ class StateView:
     entry: int
 
 
+@dataclass
+class BothView:
+    """The cache of an entry that keeps keys and values and a state."""
+    kv: KVLineView
+    state: StateView
+
+
 class Cache:
     def __init__(self, needs: Dict[int, object], readers: Dict[int, List[int]], max_tokens: int,
                  dtype: torch.dtype, device, max_slots: Optional[int] = None):
-        """``needs``: owning schedule entry -> KVNeed | StateNeed.  ``readers``: owning
+        """``needs``: owning schedule entry -> KVNeed | StateNeed | a pair of one each.  ``readers``: owning
         entry -> entries that read its cache.  ``max_tokens``: the most tokens that live
         sequences hold at any time, each sequence's count rounded up to PAGE_ROWS."""
         if max_tokens <= 0:
@@ -88,8 +96,10 @@ class Cache:
         self.states: Dict[int, torch.Tensor] = {}
         self.readers = readers
         by_key: Dict[Tuple, List[int]] = {}
-        for e in sorted(needs):
-            need = needs[e]
+        for e, need in [(e, n) for e in sorted(needs) for n in (needs[e] if isinstance(needs[e], tuple) else (needs[e],))]:
+            if isinstance(need, (KVNeed, StateNeed)) and (e in self.states if isinstance(need, StateNeed)
+                                                          else any(e in es for es in by_key.values())):
+                raise TypeError(f"schedule entry {e}: a pair of cache needs is one KVNeed and one StateNeed, got {needs[e]!r}")
             if isinstance(need, KVNeed):
                 by_key.setdefault((need.n_kv_heads, need.head_dim, need.window, need.values), []).append(e)
             elif isinstance(need, StateNeed):
@@ -221,6 +231,8 @@ class Cache:
                           owner=(entry == owner_entry), shared=bool(self.readers.get(owner_entry)))
 
     def view(self, entry: int, owner_entry: int):
+        if owner_entry in self.entry_group and owner_entry in self.states:
+            return BothView(self.line(entry, owner_entry), StateView(self.states[owner_entry], owner_entry))
         if owner_entry in self.entry_group:
             return self.line(entry, owner_entry)
         if owner_entry in self.states:

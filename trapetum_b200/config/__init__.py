@@ -5,7 +5,8 @@ from .fibelix import FibelixConfig
 from .fidepel import FidepelConfig
 from .gemma2 import Gemma2Config
 from .lofirax import LofiraxConfig
+from .ranilix import RanilixConfig
 
-__all__ = ["ArchitectureEntry", "ConfigError", "DivanexConfig", "FibelixConfig", "FidepelConfig", "Gemma2Config", "LayerSpec", "LofiraxConfig", "ModelSpec", "PartSpec", "ScheduleEntry",
+__all__ = ["ArchitectureEntry", "ConfigError", "DivanexConfig", "FibelixConfig", "FidepelConfig", "Gemma2Config", "LayerSpec", "LofiraxConfig", "ModelSpec", "PartSpec", "RanilixConfig", "ScheduleEntry",
            "architecture", "architecture_name", "known_architectures", "load_config", "read_config_dict",
            "register_architecture"]

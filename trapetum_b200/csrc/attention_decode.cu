@@ -41,6 +41,14 @@ __device__ __forceinline__ int tb_first_key(int window, int len) {
     return 0;
 }
 
+// What a weighted sum at reference M is divided by: L, or with a sink (a.sink) L + exp(sink - M).  When the sink stands far
+// above every score the quotient is taken at the sink instead, so that nothing overflows.
+__device__ __forceinline__ float tb_divided(float acc, float L, float M, const float* sink, int h) {
+    if (sink == nullptr) return acc / L;
+    const float s = sink[h], top = fmaxf(M, s), f = __expf(M - top);
+    return acc * f / (L * f + __expf(s - top));
+}
+
 template <int HD> struct DCfg {
     static constexpr int NWARP = HD >= 64 ? 16 : 8;                  // more warps hide more latency; a warp needs
     static constexpr int KPW = PAGE / NWARP;                         // at least one pass of 256 / HD keys per page
@@ -309,7 +317,7 @@ __global__ void __launch_bounds__(DCfg<HD>::NWARP * 32, 1) attn_decode_kernel(De
         }
         const int h = kvh * G + g;
         if (a.n_splits == 1) {
-            ((bf16*)a.out)[((size_t)b * a.n_heads + h) * HD + d] = __float2bfloat16_rn(acc / L);
+            ((bf16*)a.out)[((size_t)b * a.n_heads + h) * HD + d] = __float2bfloat16_rn(tb_divided(acc, L, M, a.sink, h));
         } else {
             float* p = a.partial + (((size_t)b * a.n_heads + h) * a.n_splits + split) * (HD + 2);
             p[d] = acc;
@@ -976,8 +984,8 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                     bf16* dst = (bf16*)a.out + ((size_t)b * a.n_heads + kvh * G + hg) * HD;
 #pragma unroll
                     for (int m = 0; m < C::MT_W; m++) {
-                        dst[d0 + m * 16 + quad] = __float2bfloat16_rn(o[m][e] / L);
-                        dst[d0 + m * 16 + quad + 8] = __float2bfloat16_rn(o[m][2 + e] / L);
+                        dst[d0 + m * 16 + quad] = __float2bfloat16_rn(tb_divided(o[m][e], L, M, a.sink, kvh * G + hg));
+                        dst[d0 + m * 16 + quad + 8] = __float2bfloat16_rn(tb_divided(o[m][2 + e], L, M, a.sink, kvh * G + hg));
                     }
                 } else {
                     float* dst = part_of(my_part, hg);
@@ -1029,7 +1037,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                         for (int k = 0; k < 8; k++)
                             if (k0 + k < n_parts && ms[k] != -INFINITY) { const float f = __expf(ms[k] - M); L += ls[k] * f; acc += os[k] * f; }
                     }
-                    ((bf16*)a.out)[((size_t)b * a.n_heads + kvh * G + hg) * HD + d] = __float2bfloat16_rn(acc / L);
+                    ((bf16*)a.out)[((size_t)b * a.n_heads + kvh * G + hg) * HD + d] = __float2bfloat16_rn(tb_divided(acc, L, M, a.sink, kvh * G + hg));
                 }
             }
             if (!meet(1, meet_phase)) break;                        // s_last is rewritten by the next run
@@ -1080,7 +1088,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                         for (int e = 0; e < 2; e++) { f[e] = (m[e] == -INFINITY) ? 0.f : __expf(m[e] - M); L += f[e] * l[e]; }
 #pragma unroll
                         for (int o = 16; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
-                        const float inv = 1.f / L;
+                        const float inv = tb_divided(1.f, L, M, a.sink, kvh * G + warp);
 #pragma unroll
                         for (int e = 0; e < 2; e++) wts[warp * 64 + lane + 32 * e] = f[e] * inv;
                     }
@@ -1158,7 +1166,8 @@ static int launch_mma(const DecodeArgs& a, int batch, int n_ctas, cudaStream_t s
 }
 
 // out[b,h,:] = sum_s e^(m_s - M) o_s / sum_s e^(m_s - M) l_s, splits in ascending order.
-__global__ void attn_combine_kernel(const float* __restrict__ partial, bf16* __restrict__ out, int n_splits, int hd) {
+__global__ void attn_combine_kernel(const float* __restrict__ partial, bf16* __restrict__ out, int n_splits, int hd,
+                                    const float* __restrict__ sink, int n_heads) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t bh = blockIdx.x;
@@ -1176,7 +1185,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ partial, bf16* __r
             const float ms = p[(size_t)s * (hd + 2) + hd];
             if (ms != -INFINITY) o += p[(size_t)s * (hd + 2) + d] * __expf(ms - M);
         }
-        out[bh * hd + d] = __float2bfloat16_rn(o / L);
+        out[bh * hd + d] = __float2bfloat16_rn(tb_divided(o, L, M, sink, (int)(bh % n_heads)));
     }
 }
 
@@ -1270,7 +1279,7 @@ static int run_decode(const DecodeArgs* args, int dtype, int batch, bool tensor_
     }
     if (st) return st;
     if (a.n_splits > 1 && !(tensor_cores && a.tickets != nullptr)) {
-        tb_launch(attn_combine_kernel, dim3((unsigned)batch * a.n_heads), dim3(128), 0, stream, a.partial, (bf16*)a.out, a.n_splits, a.hd);
+        tb_launch(attn_combine_kernel, dim3((unsigned)batch * a.n_heads), dim3(128), 0, stream, a.partial, (bf16*)a.out, a.n_splits, a.hd, a.sink, a.n_heads);
         st = tb_launch_status();
     }
     return st;

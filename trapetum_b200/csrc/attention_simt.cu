@@ -134,6 +134,14 @@ __global__ void attn_prefill_simt_kernel(const T* __restrict__ q, const T* __res
 // ---------------------------------------------------------------------------
 #include "decode_args.h"
 
+// What a weighted sum at reference M is multiplied with: 1 / L, or with a sink 1 / (L + exp(sink - M)) without overflow.
+__device__ __forceinline__ float inv_denominator(float M, float L, const float* sink, int h) {
+    if (sink == nullptr) return 1.f / L;
+    const float top = fmaxf(M, sink[h]);
+    const float f = expf(M - top);
+    return f / (L * f + expf(sink[h] - top));
+}
+
 template <typename T, int NC>
 __global__ void attn_decode_simt_kernel(DecodeArgs a) {
     pdl_launch_dependents();
@@ -192,7 +200,7 @@ __global__ void attn_decode_simt_kernel(DecodeArgs a) {
             if (mw != -INFINITY) o += red[(size_t)w * (hd + 2) + d] * expf(mw - M);
         }
         if (a.n_splits == 1) {
-            ((T*)a.out)[((size_t)b * a.n_heads + h) * hd + d] = from_f<T>(o / L);
+            ((T*)a.out)[((size_t)b * a.n_heads + h) * hd + d] = from_f<T>(a.sink ? o * inv_denominator(M, L, a.sink, h) : o / L);
         } else {
             a.partial[(((size_t)b * a.n_heads + h) * a.n_splits + split) * (hd + 2) + d] = o;
         }
@@ -206,7 +214,7 @@ __global__ void attn_decode_simt_kernel(DecodeArgs a) {
 // out[b,h,:] = sum_s e^(m_s - M) o_s / sum_s e^(m_s - M) l_s, splits in ascending order.
 template <typename T>
 __global__ void attn_combine_kernel(const float* __restrict__ partial, T* __restrict__ out,
-                                    int n_splits, int hd) {
+                                    int n_splits, int hd, const float* __restrict__ sink, int n_heads) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t bh = blockIdx.x;
@@ -224,7 +232,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ partial, T* __rest
             const float ms = p[(size_t)s * (hd + 2) + hd];
             if (ms != -INFINITY) o += p[(size_t)s * (hd + 2) + d] * expf(ms - M);
         }
-        out[bh * hd + d] = from_f<T>(o / L);
+        out[bh * hd + d] = from_f<T>(sink ? o * inv_denominator(M, L, sink, (int)(bh % n_heads)) : o / L);
     }
 }
 
@@ -306,7 +314,7 @@ extern "C" int tb_attn_decode_simt(const DecodeArgs* args, int dtype, int batch,
     if (a.n_splits > 1) {
         const unsigned rows = (unsigned)batch * a.n_heads;
         TB_DISPATCH_1(dtype, T,
-            tb_launch(attn_combine_kernel<T>, dim3(rows), dim3(128), 0, stream, a.partial, (T*)a.out, a.n_splits, hd));
+            tb_launch(attn_combine_kernel<T>, dim3(rows), dim3(128), 0, stream, a.partial, (T*)a.out, a.n_splits, hd, a.sink, a.n_heads));
         st = tb_launch_status();
     }
     return st;

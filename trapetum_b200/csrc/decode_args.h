@@ -44,9 +44,11 @@ typedef struct DecodeArgs {
     long long qkv_split_stride, qkv_row_stride;
     const float* inv_freq;      /* [rotary_dim / 2] */
     int rotary_dim;
+    const float* sink;          /* [n_heads] or null: head h's softmax denominator also holds exp(sink[h]), a sink
+                                   without a key and without a value */
 } DecodeArgs;
 
-#define TB_DECODE_ARGS_BYTES 168
+#define TB_DECODE_ARGS_BYTES 176
 
 #ifdef __cplusplus
 }

@@ -10,7 +10,9 @@
 //   tb_gla_scan       the recurrence; the state S of every sequence lives in a 32-bit row addressed by
 //                     slot, is read at the start of the step's tokens and written back at their end,
 //                     so a step of whole prompts and a step of one token each are the same kernel
-//   tb_gla_gate_norm  the unit norm, the weight and the gate; output in the activations' dtype
+//   tb_gla_gate_norm  the unit norm, the weight (if any) and the gate; output in the activations' dtype
+//
+// With head_decay the decay is a constant per head (retention); there is then no decay matrix and no tb_gla_decay.
 //
 // 32-bit throughout: z, the decay, the state, o and the norm.  q, k, v and g arrive in the activations'
 // dtype (they are products) and are widened on the way in.
@@ -40,7 +42,11 @@ struct GlaArgs {
     float* chunk_state;                               // [batch][n_chunks][H*D*V]: a chunk's end state from zero, then its start state
     float* chunk_decay;                               // [batch][n_chunks][H*D]: the product of the chunk's decays
     int chunk_len, n_chunks;
+    const float* head_decay;                          // [H] or null: the decay of every key channel and token of a head
 };
+
+// The argument block's size, for the Python mirror's check.
+extern "C" int tb_gla_args_bytes() { return (int)sizeof(GlaArgs); }
 
 constexpr int GLA_DECAY_TOK = 32;
 
@@ -133,7 +139,7 @@ __global__ void __launch_bounds__(GLA_WARPS * 32, 2) gla_scan_kernel(GlaArgs a) 
                 const T* row = proj + (size_t)(t0 + tt) * a.proj_stride;
                 if (MODE != 1) rq[u] = to_f<T>(row[h * D + d]) * a.q_scale;
                 rk[u] = to_f<T>(row[HD + h * D + d]);
-                rd[u] = a.decay[(size_t)(t0 + tt) * HD + h * D + d];
+                rd[u] = a.head_decay != nullptr ? a.head_decay[h] : a.decay[(size_t)(t0 + tt) * HD + h * D + d];
             }
         }
 #pragma unroll
@@ -256,7 +262,7 @@ __global__ void gla_fold_kernel(GlaArgs a) {
     }
 }
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void gla_gate_norm_kernel(GlaArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -270,15 +276,15 @@ __global__ void gla_gate_norm_kernel(GlaArgs a) {
     for (int v = lane; v < V; v += 32) sq = fmaf(y[v], y[v], sq);
     const float r = 1.f / sqrtf(warp_sum(sq) / (float)V + a.eps);
     const T* g = (const T*)a.proj + (size_t)t * a.proj_stride + 2 * HD + HV + (size_t)h * V;
-    T* o = (T*)a.out + (size_t)t * HV + (size_t)h * V;
+    TO* o = (TO*)a.out + (size_t)t * HV + (size_t)h * V;
     for (int v = lane; v < V; v += 32) {
         const float gv = to_f<T>(g[v]);
-        o[v] = from_f<T>(y[v] * r * a.norm_w[v] * (gv / (1.f + expf(-gv))));
+        o[v] = from_f<TO>(y[v] * r * (a.norm_w != nullptr ? a.norm_w[v] : 1.f) * (gv / (1.f + expf(-gv))));
     }
 }
 
 static int check(const GlaArgs& a) {
-    if (a.heads <= 0 || a.D <= 0 || a.V <= 0 || a.rank <= 0) return tb_refuse("gla: heads=%d D=%d V=%d rank=%d", a.heads, a.D, a.V, a.rank);
+    if (a.heads <= 0 || a.D <= 0 || a.V <= 0 || (a.rank <= 0 && a.head_decay == nullptr)) return tb_refuse("gla: heads=%d D=%d V=%d rank=%d", a.heads, a.D, a.V, a.rank);
     if (a.D > 256) return tb_refuse("gla: %d key channels per head; the scan keeps up to 256", a.D);
     if (a.heads > 65535 || a.batch > 65535) return tb_refuse("gla: %d heads x %d sequences exceed one launch", a.heads, a.batch);
     return 0;
@@ -341,10 +347,15 @@ extern "C" int tb_gla_plan(int heads, int V, int batch, int max_seq_len, int sms
     return (max_seq_len + len - 1) / len;
 }
 
-extern "C" int tb_gla_gate_norm(const GlaArgs* args, int dtype, cudaStream_t stream) {
+// dtype: of the gate's columns; out_dtype: of the output.
+extern "C" int tb_gla_gate_norm(const GlaArgs* args, int dtype, int out_dtype, cudaStream_t stream) {
     if (args->n_tokens <= 0) return 0;
     if (check(*args)) return -1;
     const long long items = (long long)args->n_tokens * args->heads;
-    TB_DISPATCH_1(dtype, T, tb_launch(gla_gate_norm_kernel<T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, *args));
+    if (dtype == out_dtype) {
+        TB_DISPATCH_1(dtype, T, tb_launch(gla_gate_norm_kernel<T, T>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, *args));
+    } else if (dtype == TB_F32 && out_dtype == TB_BF16) {
+        tb_launch(gla_gate_norm_kernel<float, bf16>, dim3((unsigned)((items + 3) / 4)), dim3(128), 0, stream, *args);
+    } else return tb_refuse("gla: gate dtype %d, output dtype %d", dtype, out_dtype);
     return tb_launch_status();
 }

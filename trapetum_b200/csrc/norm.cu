@@ -12,6 +12,7 @@
 //   tb_rmsnorm      out = norm(x)
 //   tb_add_rmsnorm  h (32-bit, in place) += norm_a(a);  then, if asked, out = norm_b(h);
 //                   a may be given as split-K partial sums, added here in split order
+//   tb_add_terms_rmsnorm  h += sum of up to three scaled branches;  then up to two norms of h
 //
 // Any row width works (loops are strided by the block size).
 #include "common.cuh"
@@ -622,6 +623,99 @@ extern "C" int tb_add_scaled_rmsnorm(float* h, float scale, const float* a, int 
                 h, scale, a, a_splits, a_stride, b, b_splits, b_stride, (const TW*)w, eps, offset, (TO*)out, width, row_cache))
     if (vec) ADDS(4); else ADDS(1);
 #undef ADDS
+    return tb_launch_status();
+}
+
+// Up to three branches, each with a scale of its own, added to the stream, and up to two norms of the new stream (they
+// share its root mean square) in the same pass: arrangements whose sublayers read the same stream through norms of
+// their own, and mixers whose output is a weighted sum of several products.
+//
+//   h <- h + sum_k scale_k * branch_k      branch_k: 32-bit [rows][width] or split-K partial sums; none at all: h stays
+//   out_1 = h * r * (offset + w1),  out_2 = h * r * (offset + w2),   r = 1 / sqrt(mean(h^2) + eps)
+struct AddTermsArgs {
+    float* h;
+    const float* term[3]; int splits[3]; long long stride[3]; float scale[3];
+    int n_terms;
+    const void* w1; const void* w2; void* out1; void* out2;      // w2, out2 may be null; all null: the sum alone
+    float eps, offset;
+    int rows, width;
+};
+
+// The argument block's size, for the Python mirror's check.
+extern "C" int tb_add_terms_args_bytes() { return (int)sizeof(AddTermsArgs); }
+
+template <typename TW, typename TO, int VEC>
+__global__ void __launch_bounds__(1024) add_terms_rmsnorm_kernel(AddTermsArgs a, int row_cache) {
+    pdl_launch_dependents();
+    pdl_wait();
+    extern __shared__ __align__(16) float row[];
+    __shared__ float red[33];
+    const int width = a.width;
+    const size_t base = (size_t)blockIdx.x * width;
+    float* h = a.h + base;
+    const int step = blockDim.x * VEC;
+    float ss = 0.f;
+    for (int i = threadIdx.x * VEC; i < width; i += step) {
+        float v[VEC], u[3][VEC];
+        if (VEC == 4) Vec4<float>::load(h + i, v); else v[0] = h[i];
+#pragma unroll
+        for (int k = 0; k < 3; k++) if (k < a.n_terms) load_sum<float, VEC>(a.term[k] + base + i, a.splits[k], a.stride[k], u[k]);
+#pragma unroll
+        for (int k = 0; k < 3; k++)
+            if (k < a.n_terms) {
+#pragma unroll
+                for (int e = 0; e < VEC; e++) v[e] = fmaf(a.scale[k], u[k][e], v[e]);
+            }
+#pragma unroll
+        for (int e = 0; e < VEC; e++) { ss += v[e] * v[e]; if (row_cache) row[i + e] = v[e]; }
+        if (a.n_terms > 0) { if (VEC == 4) Vec4<float>::store(h + i, v); else h[i] = v[0]; }
+    }
+    if (a.out1 == nullptr) return;
+    ss = block_sum(ss, red);
+    const float r = 1.0f / sqrtf(ss / (float)width + a.eps);
+    for (int i = threadIdx.x * VEC; i < width; i += step) {
+        float v[VEC], g[VEC], y[VEC];
+        if (row_cache) {
+#pragma unroll
+            for (int e = 0; e < VEC; e++) v[e] = row[i + e];
+        } else {
+            if (VEC == 4) Vec4<float>::load(h + i, v); else v[0] = h[i];                    // written by this thread
+        }
+        if (VEC == 4) Vec4<TW>::load((const TW*)a.w1 + i, g); else g[0] = to_f<TW>(((const TW*)a.w1)[i]);
+#pragma unroll
+        for (int e = 0; e < VEC; e++) y[e] = v[e] * r * (a.offset + g[e]);
+        TO* o1 = (TO*)a.out1 + base;
+        if (VEC == 4) Vec4<TO>::store(o1 + i, y); else o1[i] = from_f<TO>(y[0]);
+        if (a.out2 != nullptr) {
+            if (VEC == 4) Vec4<TW>::load((const TW*)a.w2 + i, g); else g[0] = to_f<TW>(((const TW*)a.w2)[i]);
+#pragma unroll
+            for (int e = 0; e < VEC; e++) y[e] = v[e] * r * (a.offset + g[e]);
+            TO* o2 = (TO*)a.out2 + base;
+            if (VEC == 4) Vec4<TO>::store(o2 + i, y); else o2[i] = from_f<TO>(y[0]);
+        }
+    }
+}
+
+extern "C" int tb_add_terms_rmsnorm(const AddTermsArgs* args, int w_dtype, int out_dtype, cudaStream_t stream) {
+    const AddTermsArgs a = *args;
+    if (a.rows <= 0) return 0;
+    if (a.width <= 0) return tb_refuse("add_terms_rmsnorm: width=%d", a.width);
+    if (!code_ok(w_dtype) || !code_ok(out_dtype)) return tb_refuse("add_terms_rmsnorm: unknown dtype codes %d %d", w_dtype, out_dtype);
+    if (a.n_terms < 0 || a.n_terms > 3) return tb_refuse("add_terms_rmsnorm: %d terms, takes up to 3", a.n_terms);
+    bool vec = a.width % 4 == 0 && aligned16(a.h) && aligned16(a.w1) && aligned16(a.w2) && aligned16(a.out1) && aligned16(a.out2);
+    for (int k = 0; k < a.n_terms; k++) {
+        if (a.term[k] == nullptr || a.splits[k] < 1) return tb_refuse("add_terms_rmsnorm: term %d is missing", k);
+        vec = vec && aligned16(a.term[k]) && a.stride[k] % 4 == 0;
+    }
+    if ((a.out1 != nullptr) != (a.w1 != nullptr) || (a.out2 != nullptr) != (a.w2 != nullptr) || (a.out2 != nullptr && a.out1 == nullptr))
+        return tb_refuse("add_terms_rmsnorm: a norm needs its weight and its output, and a second one needs a first");
+    const int row_cache = (size_t)a.width * sizeof(float) <= 40 * 1024;
+    const size_t smem = row_cache ? (size_t)a.width * sizeof(float) : 0;
+#define ADDT(VEC_)                                                                                                  \
+        DISPATCH3(TB_F32, w_dtype, out_dtype,                                                                       \
+            tb_launch(add_terms_rmsnorm_kernel<TW, TO, VEC_>, dim3(a.rows), dim3(norm_threads(a.width, VEC_)), smem, stream, a, row_cache))
+    if (vec) ADDT(4); else ADDT(1);
+#undef ADDT
     return tb_launch_status();
 }
 

@@ -78,6 +78,13 @@ def _check(lib, status: int, what: str, kernels: int = 1) -> None:
                       f"({torch.cuda.get_device_name() if torch.cuda.is_available() else 'no device'})")
 
 
+def args_mirrors():
+    """(library, function that returns the C side's size, Python structure) of the argument blocks that have such a
+    function: a mirror that has drifted from its C struct makes a kernel read garbage pointers."""
+    return (("gla", "tb_gla_args_bytes", _GlaArgs), ("retention", "tb_retention_args_bytes", _RetentionArgs),
+            ("projnorm_kv", "tb_projnorm_kv_args_bytes", _ProjNormKvArgs), ("norm", "tb_add_terms_args_bytes", _AddTermsArgs))
+
+
 def _rows_contig(t: torch.Tensor, what: str) -> None:
     if t.dim() != 2 or t.stride(1) != 1:
         raise KernelError(f"{what} must be 2-D with contiguous rows, got shape {tuple(t.shape)} strides {t.stride()}")
@@ -247,6 +254,42 @@ def add_scaled_rmsnorm(h: torch.Tensor, branches, scale: float, w: Optional[torc
                                           c_float(offset), _ptr(out), c_int(code(out_dtype) if out is not None else 0),
                                           c_int(h.shape[0]), c_int(h.shape[1]), _stream()), "add_scaled_rmsnorm")
     return out
+
+
+class _AddTermsArgs(ctypes.Structure):
+    _fields_ = [("h", c_void_p), ("term", c_void_p * 3), ("splits", c_int * 3), ("stride", c_longlong * 3), ("scale", c_float * 3),
+                ("n_terms", c_int), ("w1", c_void_p), ("w2", c_void_p), ("out1", c_void_p), ("out2", c_void_p),
+                ("eps", c_float), ("offset", c_float), ("rows", c_int), ("width", c_int)]
+
+
+def add_terms_rmsnorm(h: torch.Tensor, terms, weights=(), eps: float = 0.0, offset: float = 0.0,
+                      out_dtype: Optional[torch.dtype] = None):
+    """``h += sum of scale * branch`` in place over up to three ``terms`` (branch, scale), each branch float32 [rows,
+    width] or [splits, rows, width] partial sums; then, for up to two ``weights``, ``norm(h) * (offset + w)`` in
+    ``out_dtype`` (the norms share h's root mean square).  Returns the list of normed matrices."""
+    _cuda(h, *[t for t, _ in terms], *weights)
+    if h.dtype != torch.float32 or h.dim() != 2 or not h.is_contiguous():
+        raise KernelError("add_terms_rmsnorm: the residual stream must be contiguous float32 [rows, width]")
+    if len(terms) > 3 or len(weights) > 2:
+        raise KernelError(f"add_terms_rmsnorm: {len(terms)} terms and {len(weights)} norms; it takes up to 3 and 2")
+    a = _AddTermsArgs()
+    a.h = h.data_ptr(); a.n_terms = len(terms); a.eps = eps; a.offset = offset; a.rows = h.shape[0]; a.width = h.shape[1]
+    for k, (t, s) in enumerate(terms):
+        b, n, stride = _branch(h, t, "add_terms_rmsnorm")
+        a.term[k] = b.data_ptr(); a.splits[k] = n; a.stride[k] = stride; a.scale[k] = float(s)
+    outs = []
+    for w in weights:
+        if w.numel() != h.shape[1] or not w.is_contiguous() or w.dtype != weights[0].dtype:
+            raise KernelError("add_terms_rmsnorm: the norm weights must fit the row width and share their dtype")
+        outs.append(torch.empty(h.shape, dtype=out_dtype, device=h.device))
+    if outs:
+        a.w1 = weights[0].data_ptr(); a.out1 = outs[0].data_ptr()
+    if len(outs) == 2:
+        a.w2 = weights[1].data_ptr(); a.out2 = outs[1].data_ptr()
+    lib = build.load("norm")
+    _check(lib, lib.tb_add_terms_rmsnorm(ctypes.byref(a), c_int(code(weights[0].dtype) if outs else 0),
+                                         c_int(code(out_dtype) if outs else 0), _stream()), "add_terms_rmsnorm")
+    return outs
 
 
 def cast(x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
@@ -487,7 +530,8 @@ class _ProjNormKvArgs(ctypes.Structure):
                 ("rotary_dim", c_int), ("inv_freq", c_void_p),
                 ("positions", c_void_p), ("token_seq", c_void_p), ("len_after", c_void_p),
                 ("k_pool", c_void_p), ("v_pool", c_void_p), ("page_table", c_void_p), ("pt_stride", c_int),
-                ("page_rows", c_int), ("ring_rows", c_int), ("bias", c_void_p)]
+                ("page_rows", c_int), ("ring_rows", c_int), ("bias", c_void_p), ("head_norm", c_int), ("v_first", c_void_p),
+                ("v_lam", c_float), ("v_keep", c_void_p)]
 
 
 def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, vdim: int, padded: int,
@@ -495,7 +539,8 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
                 head_scale: Optional[torch.Tensor], rotary_dim: int, inv_freq: Optional[torch.Tensor], has_gate: bool,
                 positions: torch.Tensor, token_seq: torch.Tensor, len_after: torch.Tensor,
                 k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], page_table: Optional[torch.Tensor],
-                ring_rows: int, bias: Optional[torch.Tensor] = None):
+                ring_rows: int, bias: Optional[torch.Tensor] = None, head_norm: bool = False,
+                v_first: Optional[torch.Tensor] = None, v_lam: float = 0.0, v_keep: Optional[torch.Tensor] = None):
     """From the q/k/v(/gate) product's float32 partial sums [splits, T, H dim + G dim + G vdim (+ H)] to
     ([T, (H + 2 G) * padded] in ``out_dtype``, sigmoid of the gate columns float32 [T, H] or None): q and k divided by
     their root mean square over the whole projection times ``q_norm_w`` / ``k_norm_w`` (float32; None: no norm), q heads
@@ -503,7 +548,13 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
     token's position, every head padded with zeros to ``padded`` numbers; k and v are also written to the cache line
     (pools [pages, G, PAGE_ROWS, padded]).  ``bias``: float32, one number per column of the product (the width rounded
     up to a multiple of four), added to the summed row before anything else.  ``n_kv_heads`` 0: the product holds
-    queries only."""
+    queries only.  ``head_norm``: the norms are per head, with weights of ``dim`` numbers that the heads share.
+    ``v_first`` (float32 [T, G vdim]): the values become ``(1 - v_lam) v + v_lam v_first``; ``v_keep`` (the same shape)
+    receives this product's own values in 32-bit."""
+    _cuda(v_first, v_keep)
+    for name, t in (("v_first", v_first), ("v_keep", v_keep)):
+        if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != (partial.shape[1], n_kv_heads * vdim) or not t.is_contiguous()):
+            raise KernelError(f"projnorm_kv: {name} must be contiguous float32 [{partial.shape[1]}, {n_kv_heads * vdim}]")
     _cuda(partial, q_norm_w, k_norm_w, head_scale, inv_freq, positions, token_seq, len_after, k_pool, v_pool, page_table, bias)
     H, G = n_heads, n_kv_heads
     in_width = H * dim + G * (dim + vdim) + (H if has_gate else 0)
@@ -513,7 +564,7 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
     for name, t in (("positions", positions), ("token_seq", token_seq)):
         if t.dtype != torch.int32 or t.numel() != T or not t.is_contiguous():
             raise KernelError(f"projnorm_kv: {name} must be contiguous int32 [{T}]")
-    for name, t, n in (("q_norm_w", q_norm_w, H * dim), ("k_norm_w", k_norm_w, G * dim), ("head_scale", head_scale, H),
+    for name, t, n in (("q_norm_w", q_norm_w, dim if head_norm else H * dim), ("k_norm_w", k_norm_w, dim if head_norm else G * dim), ("head_scale", head_scale, H),
                        ("inv_freq", inv_freq, rotary_dim // 2)):
         if t is not None and (t.dtype != torch.float32 or t.numel() != n or not t.is_contiguous()):
             raise KernelError(f"projnorm_kv: {name} must be contiguous float32 [{n}]")
@@ -546,6 +597,9 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
     a.pt_stride = page_table.stride(0) if k_pool is not None else 0
     a.page_rows = PAGE_ROWS; a.ring_rows = ring_rows
     a.bias = bias.data_ptr() if bias is not None else None
+    a.head_norm = int(bool(head_norm)); a.v_lam = v_lam
+    a.v_first = v_first.data_ptr() if v_first is not None else None
+    a.v_keep = v_keep.data_ptr() if v_keep is not None else None
     lib = build.load("projnorm_kv")
     _check(lib, lib.tb_projnorm_kv(ctypes.byref(a), c_int(code(out_dtype)), c_int(T), _stream()), "projnorm_kv")
     return out, gate
@@ -562,6 +616,23 @@ def head_gate(o: torch.Tensor, gate: torch.Tensor, n_heads: int) -> torch.Tensor
     _check(lib, lib.tb_head_gate(_ptr(o), c_int(code(o.dtype)), _ptr(gate), c_int(T), c_int(n_heads),
                                  c_int(o.shape[1] // n_heads), _stream()), "head_gate")
     return o
+
+
+def value_gate(o: torch.Tensor, part: torch.Tensor, n_heads: int, value_dim: int) -> torch.Tensor:
+    """An attention output ``o`` [T, n_heads * D] times the sigmoid of ``part`` (float32 partial sums [splits, T, n_heads *
+    value_dim], added in split order), element by element; the padding beyond ``value_dim`` numbers a head is dropped:
+    returns [T, n_heads * value_dim]."""
+    _cuda(o, part)
+    T = o.shape[0]
+    if o.dim() != 2 or not o.is_contiguous() or o.shape[1] % n_heads or part.dtype != torch.float32 or part.dim() != 3 \
+            or tuple(part.shape[1:]) != (T, n_heads * value_dim) or part.stride(2) != 1:
+        raise KernelError(f"value_gate: output {tuple(o.shape)} and gate {tuple(part.shape)} do not fit {n_heads} heads of {value_dim}")
+    out = torch.empty((T, n_heads * value_dim), dtype=o.dtype, device=o.device)
+    lib = build.load("projnorm_kv")
+    _check(lib, lib.tb_value_gate(_ptr(o), _ptr(out), c_int(code(o.dtype)), _ptr(part), c_int(part.shape[0]),
+                                  c_longlong(part.stride(0)), c_longlong(part.stride(1)), c_int(T), c_int(n_heads),
+                                  c_int(o.shape[1] // n_heads), c_int(value_dim), _stream()), "value_gate")
+    return out
 
 
 def head_difference(a: torch.Tensor, n_heads: int, D: int, vdim: int, lam: float, eps: float, out_scale: float) -> torch.Tensor:
@@ -657,6 +728,12 @@ def mamba2(proj: torch.Tensor, dt_raw: torch.Tensor, heads: int, P: int, N: int,
 
 
 # ---------------------------------------------------------------------------
+def _check_sink(sink: Optional[torch.Tensor], n_heads: int) -> None:
+    _cuda(sink)
+    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != n_heads or not sink.is_contiguous()):
+        raise KernelError(f"attention: the sink must be contiguous float32 [{n_heads}]")
+
+
 def attn_prefill_simt(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, seq_start: torch.Tensor,
                       token_seq: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int,
                       scale: float, softcap: float, window: int) -> torch.Tensor:
@@ -685,14 +762,16 @@ class _DecodeArgs(ctypes.Structure):
                 ("ring_rows", c_int), ("window", c_int), ("n_splits", c_int),
                 ("scale", c_float), ("cap", c_float), ("tickets", c_void_p),
                 ("qkv_part", c_void_p), ("qkv_splits", c_int), ("qkv_split_stride", c_longlong),
-                ("qkv_row_stride", c_longlong), ("inv_freq", c_void_p), ("rotary_dim", c_int)]
+                ("qkv_row_stride", c_longlong), ("inv_freq", c_void_p), ("rotary_dim", c_int), ("sink", c_void_p)]
 
 
 def attn_decode_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                      len_after: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                      softcap: float, window: int, ring_rows: int, n_splits: int = 1,
-                     scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """One query per sequence against the paged cache (the new token's k, v already stored)."""
+                     scratch: Optional[torch.Tensor] = None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """One query per sequence against the paged cache (the new token's k, v already stored).  ``sink``: float32
+    [n_heads]; the softmax denominators then also hold ``exp(sink[h])``."""
+    _check_sink(sink, n_heads)
     _cuda(q, k_pool, v_pool, page_table, len_after, scratch)
     _rows_contig(q, "attention: q")
     B = q.shape[0]
@@ -713,6 +792,7 @@ def attn_decode_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor
     a.n_heads = n_heads; a.n_kv_heads = n_kv_heads; a.hd = head_dim; a.page_rows = PAGE_ROWS
     a.ring_rows = ring_rows; a.window = window or 0; a.n_splits = n_splits
     a.scale = scale; a.cap = softcap or 0.0
+    a.sink = sink.data_ptr() if sink is not None else None
     lib = build.load("attention_simt")
     _check(lib, lib.tb_attn_decode_simt(ctypes.byref(a), c_int(code(q.dtype)), c_int(B), _stream()), "attn_decode_simt")
     return out
@@ -1090,12 +1170,14 @@ def _set_rotation(a, part, rotate) -> None:
 def attn_decode_tma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                     len_after: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                     softcap: float, window: int, ring_rows: int, n_splits: int = 1,
-                    variant: str = "mma", rotate=None) -> torch.Tensor:
+                    variant: str = "mma", rotate=None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Decode attention with pages staged in shared memory by bulk copies (see attention_decode.cu).
     ``variant``: "mma" (tensor cores, the product path) or "lanes" (scalar, kept for comparison).
     ``rotate`` = (inv_freq or None, rotary_dim), "mma" only: ``q`` is then the float32 partial sums
     [splits, batch, (n_heads + 2 n_kv_heads) * head_dim] of the q/k/v product; the kernel adds them, rotates q and k
-    at the new token's position, and writes k and v to the cache itself (no separate rotation kernel)."""
+    at the new token's position, and writes k and v to the cache itself (no separate rotation kernel).
+    ``sink``: float32 [n_heads]; the softmax denominators then also hold ``exp(sink[h])``."""
+    _check_sink(sink, n_heads)
     _cuda(q, k_pool, v_pool, page_table, len_after)
     part = None
     if rotate is not None:
@@ -1127,6 +1209,7 @@ def attn_decode_tma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     fused_fold = variant == "mma" and head_dim >= 64 and n_splits > 1 and B * n_kv_heads <= _TICKET_SLOTS
     a.tickets = _tickets(q.device).data_ptr() if fused_fold else None
     _set_rotation(a, part, rotate)
+    a.sink = sink.data_ptr() if sink is not None else None
     lib = build.load("attention_decode")
     fn = lib.tb_attn_decode if variant == "mma" else lib.tb_attn_decode_lanes
     _check(lib, fn(ctypes.byref(a), c_int(code(q.dtype)), c_int(B), _stream()), "attn_decode",
@@ -1137,7 +1220,7 @@ def attn_decode_tma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
 def attn_decode_stream(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, page_table: torch.Tensor,
                        len_after: torch.Tensor, n_heads: int, n_kv_heads: int, head_dim: int, scale: float,
                        softcap: float, window: int, ring_rows: int, n_ctas: Optional[int] = None,
-                       rotate=None) -> torch.Tensor:
+                       rotate=None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Decode attention on tensor cores with all pages of the launch dealt out evenly to ``n_ctas`` CTAs
     (default: one per SM), wherever the sequences end: the time of a launch follows the sum of the lengths,
     not the longest one (see attention_decode.cu).  ``rotate``: as in :func:`attn_decode_tma`."""
@@ -1175,6 +1258,7 @@ def attn_decode_stream(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tens
     a.scale = scale; a.cap = softcap or 0.0
     a.tickets = _tickets(q.device).data_ptr()
     _set_rotation(a, part, rotate)
+    a.sink = sink.data_ptr() if sink is not None else None
     _check(lib, lib.tb_attn_decode_stream(ctypes.byref(a), c_int(code(q.dtype)), c_int(B), c_int(n_ctas), _stream()),
            "attn_decode_stream")
     return out
@@ -1259,26 +1343,26 @@ def attn_decode_plan(batch: int, n_kv_heads: int, len_bucket: int, ring_rows: in
 
 
 def attn_decode(q, k_pool, v_pool, page_table, len_after, n_heads, n_kv_heads, head_dim, scale, softcap, window,
-                ring_rows, len_bucket: int, uneven: int = 0, rotate=None) -> torch.Tensor:
+                ring_rows, len_bucket: int, uneven: int = 0, rotate=None, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Decode attention, kernel and partition chosen here.  ``len_bucket``: an upper bound of the longest
     context of the batch (the engine passes a power of two so that the choice is stable across steps).
     ``uneven``: how much the batch's contexts differ in length (``engine.unevenness``, 0..3); if enough, the pages
     are dealt out to the CTAs as one stream, so that the launch's time follows the sum of the lengths and not
-    the longest one."""
+    the longest one.  ``sink``: float32 [n_heads] or None, see :func:`attn_decode_tma`."""
     B = q.shape[0] if rotate is None else q.shape[1]
     dt = q.dtype if rotate is None else torch.bfloat16
     stream, splits = attn_decode_plan(B, n_kv_heads, len_bucket, ring_rows, uneven, q.device)
     if stream and attn_decode_stream_takes(dt, n_heads, n_kv_heads, head_dim, B):
         return attn_decode_stream(q, k_pool, v_pool, page_table, len_after, n_heads, n_kv_heads, head_dim, scale,
-                                  softcap, window, ring_rows, rotate=rotate)
+                                  softcap, window, ring_rows, rotate=rotate, sink=sink)
     if attn_decode_takes(dt, n_heads, n_kv_heads, head_dim):
         variant = "lanes" if head_dim < 64 else "mma"     # a 64-byte row has no swizzled box for the tensor-core kernel
         return attn_decode_tma(q, k_pool, v_pool, page_table, len_after, n_heads, n_kv_heads, head_dim, scale,
-                               softcap, window, ring_rows, splits, variant, rotate)
+                               softcap, window, ring_rows, splits, variant, rotate, sink)
     if rotate is not None:
         raise KernelError("attention: this shape's decode kernel does not rotate by itself")
     return attn_decode_simt(q, k_pool, v_pool, page_table, len_after, n_heads, n_kv_heads, head_dim, scale,
-                            softcap, window, ring_rows, splits)
+                            softcap, window, ring_rows, splits, sink=sink)
 
 
 # ---------------------------------------------------------------------------
@@ -1338,7 +1422,8 @@ class _GlaArgs(ctypes.Structure):
                 ("seq_start", c_void_p), ("token_seq", c_void_p), ("slot_ids", c_void_p),
                 ("decay", c_void_p), ("y", c_void_p), ("out", c_void_p),
                 ("heads", c_int), ("D", c_int), ("V", c_int), ("batch", c_int), ("n_tokens", c_int),
-                ("chunk_state", c_void_p), ("chunk_decay", c_void_p), ("chunk_len", c_int), ("n_chunks", c_int)]
+                ("chunk_state", c_void_p), ("chunk_decay", c_void_p), ("chunk_len", c_int), ("n_chunks", c_int),
+                ("head_decay", c_void_p)]
 
 
 def gla(proj: torch.Tensor, low: torch.Tensor, a2: torch.Tensor, a2_bias: torch.Tensor, tau: float, q_scale: float,
@@ -1378,21 +1463,86 @@ def gla(proj: torch.Tensor, low: torch.Tensor, a2: torch.Tensor, a2_bias: torch.
     a.seq_start = seq_start.data_ptr(); a.token_seq = token_seq.data_ptr(); a.slot_ids = slot_ids.data_ptr()
     a.decay = decay.data_ptr(); a.y = y.data_ptr(); a.out = out.data_ptr()
     a.heads = heads; a.D = key_dim; a.V = value_dim; a.batch = batch; a.n_tokens = T
+    a.head_decay = None
     lib = build.load("gla")
-    scan_launches = 1
+    _check(lib, lib.tb_gla_decay(ctypes.byref(a), _stream()), "gla_decay")
+    _gla_scan(lib, a, dt, max_seq_len, proj.device)
+    _check(lib, lib.tb_gla_gate_norm(ctypes.byref(a), c_int(code(dt)), c_int(code(dt)), _stream()), "gla_gate_norm")
+    return out
+
+
+def _gla_scan(lib, a, dt, max_seq_len: int, device) -> None:
+    """The recurrence of gla.cu; few long prompts are cut into chunks in time (``max_seq_len`` 0: they are not)."""
+    launches_ = 1
     if max_seq_len > 0:
         chunk_len = c_int(0)
-        n_chunks = int(lib.tb_gla_plan(c_int(heads), c_int(value_dim), c_int(batch), c_int(int(max_seq_len)),
-                                       c_int(sm_count(proj.device)), ctypes.byref(chunk_len)))
-        if n_chunks > 1 and batch * n_chunks <= 65535:
-            chunk_state = torch.empty((batch, n_chunks, HD * value_dim), dtype=torch.float32, device=proj.device)
-            chunk_decay = torch.empty((batch, n_chunks, HD), dtype=torch.float32, device=proj.device)
+        n_chunks = int(lib.tb_gla_plan(c_int(a.heads), c_int(a.V), c_int(a.batch), c_int(int(max_seq_len)),
+                                       c_int(sm_count(device)), ctypes.byref(chunk_len)))
+        if n_chunks > 1 and a.batch * n_chunks <= 65535:
+            chunk_state = torch.empty((a.batch, n_chunks, a.heads * a.D * a.V), dtype=torch.float32, device=device)
+            chunk_decay = torch.empty((a.batch, n_chunks, a.heads * a.D), dtype=torch.float32, device=device)
             a.chunk_state = chunk_state.data_ptr(); a.chunk_decay = chunk_decay.data_ptr()
             a.chunk_len = chunk_len.value; a.n_chunks = n_chunks
-            scan_launches = 3
-    _check(lib, lib.tb_gla_decay(ctypes.byref(a), _stream()), "gla_decay")
-    _check(lib, lib.tb_gla_scan(ctypes.byref(a), c_int(code(dt)), _stream()), "gla_scan", scan_launches)
-    _check(lib, lib.tb_gla_gate_norm(ctypes.byref(a), c_int(code(dt)), _stream()), "gla_gate_norm")
+            launches_ = 3
+    _check(lib, lib.tb_gla_scan(ctypes.byref(a), c_int(code(dt)), _stream()), "gla_scan", launches_)
+
+
+# ---------------------------------------------------------------------------
+# Retention
+# ---------------------------------------------------------------------------
+class _RetentionArgs(ctypes.Structure):
+    _fields_ = [("part", c_void_p), ("n_splits", c_int), ("split_stride", c_longlong), ("row_stride", c_longlong),
+                ("heads", c_int), ("D", c_int), ("V", c_int), ("rotary_dim", c_int), ("inv_freq", c_void_p),
+                ("k_scale", c_float), ("eps", c_float), ("decay", c_void_p),
+                ("positions", c_void_p), ("token_seq", c_void_p), ("seq_start", c_void_p), ("slot_ids", c_void_p),
+                ("state", c_void_p), ("state_stride", c_longlong), ("rows", c_void_p), ("out", c_void_p),
+                ("batch", c_int), ("n_tokens", c_int)]
+
+
+def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_dtype: torch.dtype, rotary_dim: int,
+              inv_freq: Optional[torch.Tensor], k_scale: float, decay: torch.Tensor, eps: float, state: torch.Tensor,
+              positions: torch.Tensor, seq_start: torch.Tensor, token_seq: torch.Tensor, slot_ids: torch.Tensor, batch: int,
+              max_seq_len: int = 0) -> torch.Tensor:
+    """Retention between its products (see retention.cu).  ``part``: float32 partial sums [splits, T, >= 2 H D + 2 H V] of
+    the input product, columns q, k, v and the gate; ``decay`` float32 [H]; ``state`` float32 [slots, H D V], rows picked
+    by ``slot_ids``, read and written.  ``max_seq_len``: the longest sequence of a step of whole prompts, 0 for a step
+    of one token each.  Returns [T, H V] in ``out_dtype``."""
+    _cuda(part, inv_freq, decay, state, positions, seq_start, token_seq, slot_ids)
+    HD, HV = heads * key_dim, heads * value_dim
+    if part.dtype != torch.float32 or part.dim() != 3 or part.stride(2) != 1 or part.shape[2] < 2 * HD + 2 * HV:
+        raise KernelError(f"retention: wants float32 partial sums [splits, tokens, >= {2 * HD + 2 * HV}], got {tuple(part.shape)} {part.dtype}")
+    T = part.shape[1]
+    if rotary_dim and (inv_freq is None or inv_freq.dtype != torch.float32 or inv_freq.numel() != rotary_dim // 2 or not inv_freq.is_contiguous()):
+        raise KernelError("retention: a rotation needs its contiguous float32 table [rotary_dim / 2]")
+    if decay.dtype != torch.float32 or decay.numel() != heads or not decay.is_contiguous():
+        raise KernelError(f"retention: the decays must be contiguous float32 [{heads}]")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] != HD * value_dim:
+        raise KernelError(f"retention: the state must be float32 [slots, {HD * value_dim}]")
+    for name, t, n in (("positions", positions, T), ("token_seq", token_seq, T), ("seq_start", seq_start, batch + 1), ("slot_ids", slot_ids, batch)):
+        if t.dtype != torch.int32 or t.numel() != n or not t.is_contiguous():
+            raise KernelError(f"retention: {name} must be contiguous int32 [{n}]")
+    out = torch.empty((T, HV), dtype=out_dtype, device=part.device)
+    a = _RetentionArgs()
+    a.part = part.data_ptr(); a.n_splits = part.shape[0]; a.split_stride = part.stride(0); a.row_stride = part.stride(1)
+    a.heads = heads; a.D = key_dim; a.V = value_dim; a.rotary_dim = rotary_dim
+    a.inv_freq = inv_freq.data_ptr() if rotary_dim else None
+    a.k_scale = k_scale; a.eps = eps; a.decay = decay.data_ptr()
+    a.positions = positions.data_ptr(); a.token_seq = token_seq.data_ptr(); a.seq_start = seq_start.data_ptr()
+    a.slot_ids = slot_ids.data_ptr(); a.state = state.data_ptr(); a.state_stride = state.stride(0)
+    a.out = out.data_ptr(); a.batch = batch; a.n_tokens = T
+    lib = build.load("retention")
+    rows = torch.empty((T, 2 * HD + 2 * HV), dtype=torch.float32, device=part.device)
+    y = torch.empty((T, HV), dtype=torch.float32, device=part.device)
+    a.rows = rows.data_ptr()
+    _check(lib, lib.tb_retention_prep(ctypes.byref(a), c_int(code(out_dtype)), _stream()), "retention_prep")
+    g = _GlaArgs()
+    g.proj = rows.data_ptr(); g.proj_stride = rows.stride(0); g.q_scale = 1.0; g.eps = eps
+    g.state = state.data_ptr(); g.state_stride = state.stride(0); g.seq_start = seq_start.data_ptr()
+    g.token_seq = token_seq.data_ptr(); g.slot_ids = slot_ids.data_ptr(); g.head_decay = decay.data_ptr()
+    g.y = y.data_ptr(); g.out = out.data_ptr(); g.heads = heads; g.D = key_dim; g.V = value_dim; g.batch = batch; g.n_tokens = T
+    gl = build.load("gla")
+    _gla_scan(gl, g, torch.float32, max_seq_len, part.device)
+    _check(gl, gl.tb_gla_gate_norm(ctypes.byref(g), c_int(code(torch.float32)), c_int(code(out_dtype)), _stream()), "gla_gate_norm")
     return out
 
 
@@ -1527,9 +1677,9 @@ def latent_decode(q: torch.Tensor, pool: torch.Tensor, page_table: torch.Tensor,
 
 
 def attn_prefill_sink(q, k, v, seq_start, token_seq, n_heads, head_dim, scale, sink, max_seq_len, seq_lens=None,
-                      window: int = 0) -> torch.Tensor:
-    """Causal prefill attention of packed sequences, one kv head per query head, whose softmax denominators also
-    hold ``exp(sink[h])`` (``sink`` float32 [n_heads], or None).  bfloat16 runs on the tcgen05 kernel (head sizes 64, 128,
+                      window: int = 0, n_kv_heads: Optional[int] = None) -> torch.Tensor:
+    """Causal prefill attention of packed sequences (``n_kv_heads`` None: one kv head per query head) whose softmax
+    denominators also hold ``exp(sink[h])`` (``sink`` float32 [n_heads], or None).  bfloat16 runs on the tcgen05 kernel (head sizes 64, 128,
     256, with the sequences' lengths on the host in ``seq_lens``) or the mma.sync kernel (other multiples of 16),
     everything else on the generic kernel."""
     _cuda(q, k, v, seq_start, token_seq, sink)
@@ -1537,8 +1687,8 @@ def attn_prefill_sink(q, k, v, seq_start, token_seq, n_heads, head_dim, scale, s
         _rows_contig(t, "attention: " + name)
     if k.stride(0) != v.stride(0) or k.dtype != q.dtype or v.dtype != q.dtype:
         raise KernelError("attention: k and v must share row stride and dtype with q")
-    if sink is not None and (sink.dtype != torch.float32 or sink.numel() != n_heads or not sink.is_contiguous()):
-        raise KernelError(f"attention: the sink must be contiguous float32 [{n_heads}]")
+    _check_sink(sink, n_heads)
+    kv = n_heads if n_kv_heads is None else n_kv_heads
     T = q.shape[0]
     out = torch.empty((T, n_heads * head_dim), dtype=q.dtype, device=q.device)
     aligned = all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, k, v))
@@ -1547,7 +1697,7 @@ def attn_prefill_sink(q, k, v, seq_start, token_seq, n_heads, head_dim, scale, s
         B = len(seq_lens)
         _check(lib, lib.tb_attn_prefill_tc_ex(_ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), c_longlong(k.stride(0)),
                                               _ptr(seq_start), _ptr(out), c_int(T), c_int(B), c_int(max(seq_lens)),
-                                              c_int(n_heads), c_int(n_heads), c_int(head_dim), c_float(scale), c_float(0.0),
+                                              c_int(n_heads), c_int(kv), c_int(head_dim), c_float(scale), c_float(0.0),
                                               c_int(window or 0), _ptr(sink), _stream()), "attn_prefill_tc", 2)
         return out
     if attn_prefill_takes(q.dtype, head_dim) and aligned:
@@ -1555,13 +1705,13 @@ def attn_prefill_sink(q, k, v, seq_start, token_seq, n_heads, head_dim, scale, s
         B = seq_start.numel() - 1
         _check(lib, lib.tb_attn_prefill_mma_ex(_ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), c_longlong(k.stride(0)),
                                                _ptr(seq_start), _ptr(out), c_int(B), c_int(max_seq_len), c_int(n_heads),
-                                               c_int(n_heads), c_int(head_dim), c_float(scale), c_float(0.0), c_int(window or 0),
+                                               c_int(kv), c_int(head_dim), c_float(scale), c_float(0.0), c_int(window or 0),
                                                _ptr(sink), _stream()), "attn_prefill_mma")
         return out
     lib = build.load("attention_simt")
     _check(lib, lib.tb_attn_prefill_simt_ex(_ptr(q), _ptr(k), _ptr(v), c_longlong(q.stride(0)), c_longlong(k.stride(0)),
                                             _ptr(seq_start), _ptr(token_seq), _ptr(out), c_int(code(q.dtype)), c_int(T),
-                                            c_int(n_heads), c_int(n_heads), c_int(head_dim), c_float(scale), c_float(0.0),
+                                            c_int(n_heads), c_int(kv), c_int(head_dim), c_float(scale), c_float(0.0),
                                             c_int(window or 0), _ptr(sink), _stream()), "attn_prefill_simt")
     return out
 

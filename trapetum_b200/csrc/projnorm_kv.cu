@@ -19,6 +19,13 @@
 //
 // A bias (one 32-bit number per column of the product) is added to the summed row first, if given.
 //
+// With head_norm the norms of q and k are per head: mean over the head's dim numbers, wq and wk of that size, shared
+// by the heads.  With v_first the values are mixed with those of an earlier layer for the same token, v <- (1 - lam) v +
+// lam v_first, before they are stored; with v_keep a layer's values leave in 32-bit as well, for later layers to mix in.
+//
+// tb_value_gate multiplies an attention output element by element with the sigmoid of columns of the same product, and
+// drops the heads' padding on the way.
+//
 // tb_head_gate multiplies every head of an attention output [tokens][H x D] by its token's gate, in place.
 //
 // tb_head_difference folds an attention output whose heads come in pairs (two score maps over the same values):
@@ -41,7 +48,13 @@ struct ProjNormKvArgs {
     const int* positions; const int* token_seq; const int* len_after;
     void* k_pool; void* v_pool; const int* page_table; int pt_stride; int page_rows; int ring_rows;
     const float* bias;                            // [in_width rounded up to 4] added to the summed row, or null
+    int head_norm;                                // the norms are per head; their weights have dim numbers
+    const float* v_first; float v_lam;            // [tokens][G * vdim] or null
+    float* v_keep;                                // [tokens][G * vdim] or null
 };
+
+// The argument block's size, for the Python mirror's check.
+extern "C" int tb_projnorm_kv_args_bytes() { return (int)sizeof(ProjNormKvArgs); }
 
 // Eight (four) consecutive numbers of an output row, rounded and stored with one or two wide stores.
 template <typename T> __device__ __forceinline__ void store8(T* dst, const float (&y)[8]);
@@ -75,7 +88,7 @@ template <typename T, int MODE>
 __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
     constexpr bool VEC = MODE != 0;
     pdl_launch_dependents();
-    extern __shared__ __align__(16) float row[];          // [in_width rounded up to 4] then cos[half], sin[half]
+    extern __shared__ __align__(16) float row[];          // [in_width rounded up to 4] then cos[half], sin[half], head roots [H + G]
     __shared__ float red[64];
     const int t = blockIdx.x;
     const int H = a.n_heads, G = a.n_kv_heads, dim = a.dim, vdim = a.vdim, D = a.D;
@@ -158,6 +171,20 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
         if (a.q_norm_w != nullptr) rq = 1.0f / sqrtf(tq / (float)nq + a.eps);
         if (a.k_norm_w != nullptr) rk = 1.0f / sqrtf(tk / (float)nk + a.eps);
     }
+    float* hr = sn + half;                                // one root per q head, then per k head
+    if (a.head_norm) {
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+        for (int hs = warp; hs < H + G; hs += nwarp) {
+            const float* x = row + hs * dim;              // the k heads follow the q heads in the row
+            float ss = 0.f;
+            for (int i = lane; i < dim; i += 32) ss = fmaf(x[i], x[i], ss);
+            ss = warp_sum(ss);
+            const bool on = (hs < H ? a.q_norm_w : a.k_norm_w) != nullptr;
+            if (lane == 0) hr[hs] = on ? 1.0f / sqrtf(ss / (float)dim + a.eps) : 1.f;
+        }
+        __syncthreads();
+    }
+    const int wstep = a.head_norm ? 0 : dim;              // from one head's norm weights to the next one's
     T* orow = (T*)a.out + (size_t)t * a.out_row_stride;
     const int n_qk = (H + G) * D;
     T* vrow = orow + n_qk;
@@ -175,11 +202,12 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
                 const int c0 = head * dim;
                 const float* x = row + (is_q ? 0 : nq) + c0;
                 const float* w = is_q ? a.q_norm_w : a.k_norm_w;
-                const float f = (is_q ? rq : rk) * ((is_q && a.head_scale != nullptr) ? a.head_scale[head] : 1.f);
+                const float f = (a.head_norm ? hr[hs] : is_q ? rq : rk) * ((is_q && a.head_scale != nullptr) ? a.head_scale[head] : 1.f);
+                const int w0 = head * wstep;
                 float4 xi = *(const float4*)(x + i0);
                 xi.x *= f; xi.y *= f; xi.z *= f; xi.w *= f;
                 if (w != nullptr) {
-                    const float4 wi = __ldg((const float4*)(w + c0 + i0));
+                    const float4 wi = __ldg((const float4*)(w + w0 + i0));
                     xi.x *= wi.x; xi.y *= wi.y; xi.z *= wi.z; xi.w *= wi.w;
                 }
                 if (i0 < R) {
@@ -188,7 +216,7 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
                     float4 xj = *(const float4*)(x + j0);
                     xj.x *= f; xj.y *= f; xj.z *= f; xj.w *= f;
                     if (w != nullptr) {
-                        const float4 wj = __ldg((const float4*)(w + c0 + j0));
+                        const float4 wj = __ldg((const float4*)(w + w0 + j0));
                         xj.x *= wj.x; xj.y *= wj.y; xj.z *= wj.z; xj.w *= wj.w;
                     }
                     const float4 c = *(const float4*)(cs + a0), sv = *(const float4*)(sn + a0);
@@ -205,7 +233,13 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
         }
         for (int u = threadIdx.x; u < G * per; u += blockDim.x) {
             const int g = u / per, i0 = (u - g * per) << 2;
-            const float4 y = i0 < vdim ? *(const float4*)(row + nq + nk + g * vdim + i0) : make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 y = i0 < vdim ? *(const float4*)(row + nq + nk + g * vdim + i0) : make_float4(0.f, 0.f, 0.f, 0.f);
+            if (i0 < vdim && a.v_keep != nullptr) *(float4*)(a.v_keep + (size_t)t * nv + g * vdim + i0) = y;
+            if (i0 < vdim && a.v_first != nullptr) {
+                const float4 f = *(const float4*)(a.v_first + (size_t)t * nv + g * vdim + i0);
+                const float m = 1.f - a.v_lam;
+                y.x = m * y.x + a.v_lam * f.x; y.y = m * y.y + a.v_lam * f.y; y.z = m * y.z + a.v_lam * f.z; y.w = m * y.w + a.v_lam * f.w;
+            }
             store4<T>(vrow + (size_t)g * D + i0, y);
             if (store) store4<T>((T*)a.v_pool + (cache_row + (size_t)g * a.page_rows) * D + i0, y);
         }
@@ -220,11 +254,12 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
                 const int c0 = head * dim;                                               // the head's first column in its projection
                 const float* x = row + (is_q ? 0 : nq);
                 const float* w = is_q ? a.q_norm_w : a.k_norm_w;
-                const float f = (is_q ? rq : rk) * ((is_q && a.head_scale != nullptr) ? a.head_scale[head] : 1.f);
-                const float xi = x[c0 + i] * (w != nullptr ? w[c0 + i] : 1.f) * f;
+                const float f = (a.head_norm ? hr[hs] : is_q ? rq : rk) * ((is_q && a.head_scale != nullptr) ? a.head_scale[head] : 1.f);
+                const int w0 = head * wstep;
+                const float xi = x[c0 + i] * (w != nullptr ? w[w0 + i] : 1.f) * f;
                 if (i < R) {
                     const int j = i < half ? i + half : i - half, ai = i < half ? i : i - half;
-                    const float xj = x[c0 + j] * (w != nullptr ? w[c0 + j] : 1.f) * f;
+                    const float xj = x[c0 + j] * (w != nullptr ? w[w0 + j] : 1.f) * f;
                     y = i < half ? xi * cs[ai] - xj * sn[ai] : xi * cs[ai] + xj * sn[ai];
                 } else {
                     y = xi;
@@ -237,7 +272,10 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
         // v heads: as they are, padded
         for (int e = threadIdx.x; e < G * D; e += blockDim.x) {
             const int g = e / D, i = e - g * D;
-            const T yy = from_f<T>(i < vdim ? row[nq + nk + g * vdim + i] : 0.f);
+            float y = i < vdim ? row[nq + nk + g * vdim + i] : 0.f;
+            if (i < vdim && a.v_keep != nullptr) a.v_keep[(size_t)t * nv + g * vdim + i] = y;
+            if (i < vdim && a.v_first != nullptr) y = (1.f - a.v_lam) * y + a.v_lam * a.v_first[(size_t)t * nv + g * vdim + i];
+            const T yy = from_f<T>(y);
             vrow[e] = yy;
             if (store) ((T*)a.v_pool)[(cache_row + (size_t)g * a.page_rows) * D + i] = yy;
         }
@@ -260,7 +298,7 @@ extern "C" int tb_projnorm_kv(const ProjNormKvArgs* args, int out_dtype, int n_t
     if (a.ring_rows > 0 && a.ring_rows % a.page_rows != 0)
         return tb_refuse("projnorm_kv: ring_rows=%d must be a multiple of page_rows=%d", a.ring_rows, a.page_rows);
     const long long in_width = (long long)a.n_heads * a.dim + (long long)a.n_kv_heads * (a.dim + a.vdim) + (a.gate_out ? a.n_heads : 0);
-    const size_t smem = (size_t)(((in_width + 3) & ~3LL) + a.rotary_dim) * sizeof(float);
+    const size_t smem = (size_t)(((in_width + 3) & ~3LL) + a.rotary_dim + (a.head_norm ? a.n_heads + a.n_kv_heads : 0)) * sizeof(float);
     if (smem > 200 * 1024) return tb_refuse("projnorm_kv: a projection of %lld numbers exceeds one block's shared memory", in_width);
     const int half = a.rotary_dim / 2;
     const size_t el = out_dtype == TB_BF16 ? 2 : 4;
@@ -270,7 +308,8 @@ extern "C" int tb_projnorm_kv(const ProjNormKvArgs* args, int out_dtype, int n_t
         && ((uintptr_t)a.out % 16 == 0) && (a.out_row_stride * el) % 16 == 0
         && (a.q_norm_w == nullptr || (uintptr_t)a.q_norm_w % 16 == 0) && (a.k_norm_w == nullptr || (uintptr_t)a.k_norm_w % 16 == 0)
         && (a.k_pool == nullptr || ((uintptr_t)a.k_pool % 16 == 0 && (uintptr_t)a.v_pool % 16 == 0))
-        && (a.bias == nullptr || (uintptr_t)a.bias % 16 == 0);
+        && (a.bias == nullptr || (uintptr_t)a.bias % 16 == 0)
+        && (uintptr_t)a.v_first % 16 == 0 && (uintptr_t)a.v_keep % 16 == 0;
     // few tokens (a decode step) leave most of the GPU idle and are a chain of memory waits: four times the threads a
     // token shorten the chain; many tokens fill the GPU with blocks of 256
     const int threads = n_tokens <= 2 * 148 ? 1024 : 256;
@@ -331,6 +370,53 @@ extern "C" int tb_head_gate(void* o, int dtype, const float* gate, int n_tokens,
         return tb_launch_status();
     }
     TB_DISPATCH_1(dtype, T, tb_launch(head_gate_kernel<T>, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, stream, (T*)o, gate, n, D));
+    return tb_launch_status();
+}
+
+// out[t][h * V + i] = o[t][h * D + i] * sigmoid(z[t][h * V + i]), z the sum of the partial sums [splits][tokens][..] in
+// split order.  VEC = 4: V, D and the strides are multiples of four and the rows aligned; VEC = 1: anything.
+template <typename T, int VEC>
+__global__ void value_gate_kernel(const T* __restrict__ o, T* __restrict__ out, const float* __restrict__ z, int n_splits,
+                                  long long split_stride, long long row_stride, long long n, int H, int D, int V) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long u = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+    if (u >= n) return;
+    const int HV = H * V;
+    const long long t = u / HV;
+    const int c = (int)(u - t * HV), h = c / V, i = c - h * V;
+    const float* zp = z + t * row_stride + c;
+    const T* src = o + (t * H + h) * D + i;
+    if (VEC == 4) {
+        float4 s = *(const float4*)zp;
+#pragma unroll 8
+        for (int sp = 1; sp < n_splits; sp++) {
+            const float4 x = *(const float4*)(zp + sp * split_stride);
+            s.x += x.x; s.y += x.y; s.z += x.z; s.w += x.w;
+        }
+        float v[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) v[e] = to_f<T>(src[e]);
+        store4<T>(out + u, make_float4(v[0] / (1.f + expf(-s.x)), v[1] / (1.f + expf(-s.y)), v[2] / (1.f + expf(-s.z)), v[3] / (1.f + expf(-s.w))));
+    } else {
+        float s = 0.f;
+        for (int sp = 0; sp < n_splits; sp++) s += zp[sp * split_stride];
+        out[u] = from_f<T>(to_f<T>(*src) / (1.f + expf(-s)));
+    }
+}
+
+// o [tokens][H * D] (contiguous) -> out [tokens][H * V].
+extern "C" int tb_value_gate(const void* o, void* out, int dtype, const float* z, int n_splits, long long split_stride,
+                             long long row_stride, int n_tokens, int H, int D, int V, cudaStream_t stream) {
+    const long long n = (long long)n_tokens * H * V;
+    if (n <= 0) return 0;
+    if (V > D || n_splits < 1) return tb_refuse("value_gate: values of %d in heads of %d, %d splits", V, D, n_splits);
+    const bool vec = V % 4 == 0 && D % 4 == 0 && (uintptr_t)o % 16 == 0 && (uintptr_t)out % 16 == 0 && (uintptr_t)z % 16 == 0
+        && split_stride % 4 == 0 && row_stride % 4 == 0;
+#define TB_VALUE_GATE(V_) TB_DISPATCH_1(dtype, T, tb_launch(value_gate_kernel<T, V_>, dim3((unsigned)((n / V_ + 255) / 256)), dim3(256), 0, stream, \
+        (const T*)o, (T*)out, z, n_splits, split_stride, row_stride, n, H, D, V))
+    if (vec) TB_VALUE_GATE(4); else TB_VALUE_GATE(1);
+#undef TB_VALUE_GATE
     return tb_launch_status();
 }
 

@@ -58,8 +58,22 @@ Three more options change who sees whom and how the scores become weights; they 
 * ``talk`` (a tensor name, [heads, heads]): the heads' scores are mixed before the mask and the softmax,
   ``s_h <- sum_g talk[h, g] s_g``.  Scale and ``head_temp`` are folded into the matrix when the weights are bound.
 
+Five more options of the same path, which go without ``proj_norm``, ``head_temp``, ``out_gate`` and the three above:
+
+* ``head_norm`` ``{"q": name, "k": name, "eps": e}``: every query / key head is divided by its root mean square over
+  ``head_dim`` and multiplied by a weight of that size that the heads share, before the rotation (32-bit, inside
+  ``ops.projnorm_kv``; the plain path's ``q_norm`` / ``k_norm`` run as kernels of their own);
+* ``sink`` (a tensor name, one number per head): the softmax denominator of head h also holds ``exp(sink[h])``;
+* ``v_mix`` ``{"weight": name, "first": bool, "group": key}``: the first layer of a group keeps its values for the
+  running step; the others mix them into their own, ``v <- (1 - lam) v + lam v_first`` (same token), before the cache;
+* ``value_gate`` (a tensor name, [heads * value_dim, hidden]): the concatenated heads are multiplied element by element
+  with ``sigmoid(G x)`` before the output projection; its rows ride in the fused projection;
+* a ``position`` whose pairs are neighbours: a row order of the bound q and k weights (and of what acts on their
+  heads), after which it is the rotate-half rotation (any path).
+
 The three projections are fused into one matrix when the weights are bound, so
-a step runs one product for q, k and v.
+a step runs one product for q, k and v.  A mixer that contains this one may make that product together with others
+(``in_weight``, :meth:`Attention.finish`).
 """
 from __future__ import annotations
 
@@ -128,8 +142,22 @@ class Attention(Mixer):
             raise ValueError("attention: 'block' and 'window' exclude each other")
         if self.block is not None and self.block < 1:
             raise ValueError(f"attention: block={self.block} must be positive")
+        hn = dict(p.get("head_norm") or {})
+        self.head_norm_names = {key: hn[key] for key in ("q", "k") if hn.get(key)}
+        self.sink_name = p.get("sink")
+        self.v_mix = dict(p.get("v_mix") or {})
+        self.value_gate_name = p.get("value_gate")
+        per_head = bool(self.head_norm_names or self.sink_name or self.v_mix or self.value_gate_name)
+        if per_head and (self.proj_norm_names or self.head_temp_name or self.out_gate_name or self.mixed):
+            raise ValueError("attention: 'head_norm', 'sink', 'v_mix' and 'value_gate' go without 'proj_norm', 'head_temp', "
+                             "'out_gate', 'block', 'unit_sink' and 'talk'")
+        if self.head_norm_names:
+            self.proj_norm_eps = float(hn.get("eps", 0.0))
         self.projected = bool(self.proj_norm_names or self.head_temp_name or self.out_gate_name or self.vd != self.hd
-                              or self.mixed)
+                              or self.mixed or per_head)
+        self.order = self.position.head_order()
+        if self.order is not None and (self.q_norm or self.k_norm):
+            raise ValueError("attention: 'q_norm' and 'k_norm' go with a rotation of halves; use 'head_norm'")
         if self.projected:
             if self.prepared or self.q_norm or self.k_norm or self.softcap:
                 raise ValueError("attention: 'proj_norm', 'head_temp', 'value_dim', 'out_gate', 'block', 'unit_sink' and 'talk' "
@@ -140,7 +168,8 @@ class Attention(Mixer):
             # the mixing kernels take any head size; the tensor-core kernels want one of theirs
             self.pad = ops.attn_mixed_padded_head(rt.dtype, self.n_heads, max(self.hd, self.vd)) if self.mixed \
                 else ops.attn_padded_head(rt.dtype, max(self.hd, self.vd))
-        self.wq_norm = self.wk_norm = self.head_temp = self.w_o_padded = self.mix = self.b_proj = None
+        self.wq_norm = self.wk_norm = self.head_temp = self.w_o_padded = self.mix = self.b_proj = self.sink = None
+        self.v_lam = 0.0
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         specs = {
@@ -159,6 +188,14 @@ class Attention(Mixer):
             specs[self.prefix + self.out_gate_name] = TensorSpec((self.n_heads, self.hidden))
         if self.talk_name:
             specs[self.prefix + self.talk_name] = TensorSpec((self.n_heads, self.n_heads))
+        for key in self.head_norm_names:
+            specs[self.prefix + self.head_norm_names[key]] = TensorSpec((self.hd,), "gain")
+        if self.sink_name:
+            specs[self.prefix + self.sink_name] = TensorSpec((self.n_heads,), "norm")
+        if self.v_mix.get("weight"):
+            specs[self.prefix + self.v_mix["weight"]] = TensorSpec((), "norm", optional=bool(self.v_mix.get("first")))
+        if self.value_gate_name:
+            specs[self.prefix + self.value_gate_name] = TensorSpec((self.n_heads * self.vd, self.hidden))
         sizes = {"q": self.qd, "k": self.kvd, "v": self.n_kv * self.vd, "o": self.hidden}
         for key, name in self.bias_names.items():
             specs[self.prefix + name] = TensorSpec((sizes[key],))
@@ -170,16 +207,35 @@ class Attention(Mixer):
     def bind(self, tensors) -> None:
         mats = [tensors[self._name(n)] for n in (("q", "k") if self.v_from_k else ("q", "k", "v"))]
         q = mats[0]
+        order = None if self.order is None else torch.tensor(self.order, device=q.device)
+
+        def ordered(t):
+            """The numbers of every q or k head (along the first axis) in the order that makes the rotation one of halves."""
+            return t if order is None else t.view((-1, self.hd) + tuple(t.shape[1:]))[:, order].reshape(t.shape)
+        mats[0], mats[1] = ordered(mats[0]), ordered(mats[1])
         if self.projected:
             if self.out_gate_name:
                 mats.append(tensors[self.prefix + self.out_gate_name])
+            if self.value_gate_name:
+                # from a multiple of four columns on, so that the gate's 16-byte loads are aligned
+                self.gate_col = sum(m.shape[0] for m in mats)
+                pad = -self.gate_col % 4
+                if pad:
+                    mats.append(torch.zeros((pad, self.hidden), dtype=q.dtype, device=q.device))
+                    self.gate_col += pad
+                mats.append(tensors[self.prefix + self.value_gate_name])
             n = sum(m.shape[0] for m in mats)
             mats.append(torch.zeros((-n % 16, self.hidden), dtype=q.dtype, device=q.device))     # whole tiles of weight rows
             # short vectors that enter 32-bit arithmetic: kept in 32 bits (exact for what a file stores in 16)
-            if "q" in self.proj_norm_names:
-                self.wq_norm = tensors[self.prefix + self.proj_norm_names["q"]].float().contiguous()
-            if "k" in self.proj_norm_names:
-                self.wk_norm = tensors[self.prefix + self.proj_norm_names["k"]].float().contiguous()
+            norms = self.head_norm_names or self.proj_norm_names
+            if "q" in norms:
+                self.wq_norm = ordered(tensors[self.prefix + norms["q"]].float()).contiguous()
+            if "k" in norms:
+                self.wk_norm = ordered(tensors[self.prefix + norms["k"]].float()).contiguous()
+            if self.sink_name:
+                self.sink = tensors[self.prefix + self.sink_name].float().contiguous()
+            if self.v_mix and not self.v_mix.get("first"):
+                self.v_lam = float(tensors[self.prefix + self.v_mix["weight"]].float())
             if self.head_temp_name:
                 self.head_temp = tensors[self.prefix + self.head_temp_name].float().contiguous()
             if self.mixed:
@@ -193,10 +249,11 @@ class Attention(Mixer):
                 parts = [tensors[self.prefix + self.bias_names[key]].float() if key in self.bias_names
                          else torch.zeros(m, dtype=torch.float32, device=q.device)
                          for key, m in (("q", self.qd), ("k", self.kvd), ("v", self.n_kv * self.vd))]
+                parts[0], parts[1] = ordered(parts[0]), ordered(parts[1])
                 parts.append(torch.zeros(n - sum(x.numel() for x in parts) + (-n % 16), dtype=torch.float32, device=q.device))
                 self.b_proj = torch.cat(parts).contiguous()
             w_o = tensors[self._name("o")]
-            if self.pad != self.vd:
+            if self.pad != self.vd and not self.value_gate_name:          # (the gate's kernel drops the padding)
                 wide = torch.zeros((self.hidden, self.n_heads, self.pad), dtype=w_o.dtype, device=w_o.device)
                 wide[:, :, :self.vd] = w_o.view(self.hidden, self.n_heads, self.vd)
                 w_o = wide.view(self.hidden, self.n_heads * self.pad).contiguous()
@@ -210,6 +267,7 @@ class Attention(Mixer):
             parts = [tensors[self.prefix + self.bias_names[key]].float() if key in self.bias_names
                      else torch.zeros(n, dtype=torch.float32, device=q.device)
                      for key, n in (("q", self.qd), ("k", self.kvd), ("v", self.kvd))]
+            parts[0], parts[1] = ordered(parts[0]), ordered(parts[1])
             self.b_qkv = torch.cat(parts).contiguous()
         if "o" in self.bias_names:
             self.b_o = tensors[self.prefix + self.bias_names["o"]].float().contiguous()
@@ -269,10 +327,44 @@ class Attention(Mixer):
     def cache_need(self):
         return KVNeed(self.n_kv, self.pad if self.projected else self.hd, self.block or self.window)
 
+    @property
+    def in_weight(self) -> torch.Tensor:
+        """The fused input matrix: a mixer that contains this one may make its product together with others and hand the
+        columns to :meth:`finish`."""
+        return self.w_qkv
+
+    @in_weight.setter
+    def in_weight(self, w: torch.Tensor) -> None:
+        self.w_qkv = w
+
+    def finish(self, part, ctx, line):
+        """The rest of the mixer: ``part`` is the product with ``in_weight`` as 32-bit partial sums [splits, T, width]."""
+        if self.projected:
+            return self._finish_projected(part, ctx, line)
+        if not line.owner or self.prepared or self.b_qkv is not None or self.q_norm is not None or self.k_norm is not None:
+            raise NotImplementedError("attention: 'finish' takes the plain and the projected path of a mixer that owns its cache")
+        dt, H, G, D = self.rt.dtype, self.n_heads, self.n_kv, self.hd
+        part = part[:, :, :(H + 2 * G) * D]
+        rotate = self.position.rotary_table()
+        if not ctx.is_prefill and rotate is not None and ops.attn_decode_rotates(dt, H, G, D):
+            # decoding: the attention kernel adds the partial sums up, rotates and appends to the cache by itself
+            return self._out(ops.attn_decode(part, line.k, line.v, line.page_table, ctx.len_after, H, G, D, self.scale, self.softcap,
+                                             self.window or 0, line.ring_rows, ctx.len_bucket, ctx.uneven, rotate))
+        qkv = torch.empty(part.shape[1:], dtype=dt, device=part.device)
+        self.position.rotate_and_store(qkv, H, G, ctx, line, store=True, partial=part)
+        q, k, v = qkv[:, :H * D], qkv[:, H * D:(H + G) * D], qkv[:, (H + G) * D:]
+        if ctx.is_prefill:
+            o = ops.attn_prefill(q, k, v, ctx.seq_start, ctx.token_seq, H, G, D, self.scale, self.softcap, self.window or 0,
+                                 ctx.max_seq_len, ctx.seq_lens, ctx.memo)
+        else:
+            o = ops.attn_decode(q, line.k, line.v, line.page_table, ctx.len_after, H, G, D, self.scale, self.softcap,
+                                self.window or 0, line.ring_rows, ctx.len_bucket, ctx.uneven)
+        return self._out(o)
+
     def forward(self, x, ctx, line):
         dt = self.rt.dtype
         if self.projected:
-            return self._forward_projected(x, ctx, line)
+            return self._finish_projected(linear_partials(x, self.w_qkv), ctx, line)
         if self.prepared:
             return self._forward_prepared(x, ctx, line)
         if line.owner:
@@ -337,20 +429,27 @@ class Attention(Mixer):
         return self._out(o)
 
 
-    def _forward_projected(self, x, ctx, line):
-        """The path of ``proj_norm`` / ``head_temp`` / ``value_dim`` / ``out_gate``: the fused projection as 32-bit partial
-        sums, one kernel that norms, weighs, rotates, pads, rounds, fills the cache and takes the gate's sigmoid, then the
-        same attention kernels as every other mixer at the padded head size."""
+    def _finish_projected(self, part, ctx, line):
+        """The path of ``proj_norm`` / ``head_norm`` / ``head_temp`` / ``value_dim`` / the gates / ``sink`` / ``v_mix``: the
+        fused projection as 32-bit partial sums, one kernel that norms, weighs, rotates, pads, rounds, mixes values, fills the
+        cache and takes the head gate's sigmoid, then the same attention kernels as every other mixer at the padded head
+        size, and the gate."""
         dt = self.rt.dtype
         if not line.owner:
             raise NotImplementedError("attention: a mixer with a projection-wide norm that reads another call's cache is not built")
         H, G, D = self.n_heads, self.n_kv, self.pad
         inv_freq, rotary = self.position.rotary_table()
-        part = linear_partials(x, self.w_qkv)
+        first = keep = None
+        if self.v_mix:
+            key = ("v_first", self.v_mix.get("group"))
+            if self.v_mix.get("first"):
+                keep = ctx.memo[key] = torch.empty((part.shape[1], G * self.vd), dtype=torch.float32, device=part.device)
+            else:
+                first = ctx.memo[key]
         qkv, gate = ops.projnorm_kv(part, H, G, self.hd, self.vd, D, dt, self.wq_norm, self.wk_norm, self.proj_norm_eps,
                                     None if self.mixed else self.head_temp, rotary, inv_freq, bool(self.out_gate_name),
                                     ctx.positions, ctx.token_seq, ctx.len_after, line.k, line.v, line.page_table,
-                                    line.ring_rows, self.b_proj)
+                                    line.ring_rows, self.b_proj, bool(self.head_norm_names), first, self.v_lam, keep)
         q = qkv[:, :H * D]
         k = qkv[:, H * D:(H + G) * D]
         v = qkv[:, (H + G) * D:]
@@ -362,14 +461,19 @@ class Attention(Mixer):
             else:
                 o = ops.attn_mixed_decode(q, line.k, line.v, line.page_table, ctx.len_after, H, G, D, self.mix, seen,
                                           self.unit_sink, line.ring_rows, ctx.len_bucket)
+        elif ctx.is_prefill and self.sink is not None:
+            o = ops.attn_prefill_sink(q, k, v, ctx.seq_start, ctx.token_seq, H, D, self.scale, self.sink, ctx.max_seq_len,
+                                      ctx.seq_lens, self.window or 0, n_kv_heads=G)
         elif ctx.is_prefill:
             o = ops.attn_prefill(q, k, v, ctx.seq_start, ctx.token_seq, H, G, D, self.scale, 0.0, self.window or 0,
                                  ctx.max_seq_len, ctx.seq_lens, ctx.memo)
         else:
             o = ops.attn_decode(q, line.k, line.v, line.page_table, ctx.len_after, H, G, D, self.scale, 0.0,
-                                self.window or 0, line.ring_rows, ctx.len_bucket, ctx.uneven)
+                                self.window or 0, line.ring_rows, ctx.len_bucket, ctx.uneven, sink=self.sink)
         if gate is not None:
             ops.head_gate(o, gate, H)
+        if self.value_gate_name:
+            o = ops.value_gate(o, part[:, :, self.gate_col:self.gate_col + H * self.vd], H, self.vd)
         return self._out(o)
 
 

@@ -64,6 +64,13 @@ class StateNeed:
     dtype: torch.dtype = torch.float32
 
 
+@dataclass(frozen=True)
+class Terms:
+    """A sublayer's output as a weighted sum that nobody has made yet: (branch output, scale) pairs, each branch float32
+    [tokens, hidden] or its [splits, tokens, hidden] partial sums.  The block adds them to the stream together."""
+    pairs: Tuple[Tuple[torch.Tensor, float], ...]
+
+
 # ---------------------------------------------------------------------------
 # Interfaces
 # ---------------------------------------------------------------------------
@@ -113,6 +120,12 @@ class Norm(Part):
 
 
 class PositionEncoding(Part):
+    def head_order(self):
+        """None, or the order (a list of ``head_dim`` places) in which a mixer has to lay out every q and k head's
+        numbers so that the rotation becomes the rotate-half one that the kernels apply: a rotation of other pairs is
+        a row order of the bound weights, to which no score is sensitive."""
+        return None
+
     def rotary_table(self):
         """``(inv_freq, rotary_dim)`` if this encoding is the rotate-half rotation of the first ``rotary_dim`` dims
         of q and k by ``position * inv_freq[i]`` (``(None, 0)``: it changes nothing), so that a mixer's kernel
@@ -122,15 +135,16 @@ class PositionEncoding(Part):
 
 class Mixer(Part):
     def cache_need(self):
-        """:class:`KVNeed`, :class:`StateNeed` or None."""
+        """:class:`KVNeed`, :class:`StateNeed`, a pair of one each (a mixer that keeps both), or None."""
         return None
 
     def forward(self, x: torch.Tensor, ctx, cache) -> torch.Tensor:
         """``x`` [tokens, hidden] in the compute dtype; ``ctx`` the step's
         :class:`~trapetum_b200.engine.step.StepContext`; ``cache`` this call's view
         of the cache (:class:`~trapetum_b200.cache.kv.KVLineView`, a state tensor
-        view, or None).  Returns [tokens, hidden], or [splits, tokens, hidden] float32 partial
-        sums whose sum over the first axis is the result (the residual stream adds them)."""
+        view, a :class:`~trapetum_b200.cache.kv.BothView`, or None).  Returns [tokens, hidden], or
+        [splits, tokens, hidden] float32 partial sums whose sum over the first axis is the result (the residual
+        stream adds them), or :class:`Terms` (for blocks that take them)."""
         raise NotImplementedError
 
 

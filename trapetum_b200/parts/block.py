@@ -24,7 +24,12 @@ added together, times ``scale`` (1 if absent):
 
     x = norm(h);  h += scale * (mixer(x) + feed_forward(x))
 
-(without a feed-forward: ``h += scale * mixer(x)``).
+(without a feed-forward: ``h += scale * mixer(x)``).  With ``ffn_norm`` the feed-forward reads the same stream
+through a norm of its own:
+
+    h += scale * (mixer(norm(h)) + feed_forward(ffn_norm(h)))
+
+A mixer may return :class:`~trapetum_b200.parts.base.Terms`, products that are added with a scale each.
 
 A block only talks to the :class:`~trapetum_b200.parts.stream.ResidualStream`,
 which decides how additions and norms are fused.
@@ -34,7 +39,7 @@ from __future__ import annotations
 from typing import Dict
 
 from ..weights.loader import TensorSpec
-from .base import Block, build_part, register_part
+from .base import Block, Terms, build_part, register_part
 
 
 class _NormedBlock(Block):
@@ -65,6 +70,14 @@ class _NormedBlock(Block):
         return out
 
 
+def _with_idle(block, specs: Dict[str, TensorSpec]) -> Dict[str, TensorSpec]:
+    """``idle``: tensor name -> size of vectors that a file may carry for a layer without feed-forward (the norm that
+    nothing follows); they are accepted and not used."""
+    for name, size in (block.params.get("idle") or {}).items():
+        specs.setdefault(block.prefix + name, TensorSpec((int(size),), "norm", optional=True))
+    return specs
+
+
 class SandwichBlock(_NormedBlock):
     NORMS = ("pre_mixer_norm", "post_mixer_norm", "pre_ffn_norm", "post_ffn_norm")
 
@@ -89,12 +102,7 @@ class PreNormBlock(_NormedBlock):
                       if n == "pre_mixer_norm" or self.has_ffn}
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
-        specs = super().tensor_specs()
-        # ``idle``: tensor name -> size of vectors that a file may carry for a layer without feed-forward (the norm
-        # that nothing follows); they are accepted and not used
-        for name, size in (self.params.get("idle") or {}).items():
-            specs.setdefault(self.prefix + name, TensorSpec((int(size),), "norm", optional=True))
-        return specs
+        return _with_idle(self, super().tensor_specs())
 
     def forward(self, stream, ctx, cache) -> None:
         dt = self.rt.dtype
@@ -140,19 +148,35 @@ class PostNormBlock(_NormedBlock):
 
 
 class ParallelBlock(_NormedBlock):
-    """Parameters: ``norm`` (the one norm's spec) and ``scale``."""
-    NORMS = ("norm",)
+    """Parameters: ``norm`` (the mixer's norm, and the feed-forward's unless ``ffn_norm`` is given), ``ffn_norm``
+    (optional), ``scale``, and ``idle`` (see :class:`PreNormBlock`)."""
 
     def __init__(self, params, prefix, rt, mixer, feed_forward):
-        super().__init__(params, prefix, rt, mixer, feed_forward)
+        Block.__init__(self, params, prefix, rt, mixer, feed_forward)
         self.scale = float(params.get("scale", 1.0))
         self.has_ffn = not getattr(feed_forward, "absent", False)
+        self.two_norms = self.has_ffn and bool(params.get("ffn_norm"))
+        self.norms = {n: build_part("norm", params[n], prefix, rt) for n in (("norm", "ffn_norm") if self.two_norms else ("norm",))}
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return _with_idle(self, super().tensor_specs())
 
     def forward(self, stream, ctx, cache) -> None:
-        x = stream.normed(self.norms["norm"], self.rt.dtype)
-        branches = [self.mixer.forward(x, ctx, cache)]
+        dt = self.rt.dtype
+        if self.two_norms:
+            x, x_ffn = stream.normed_pair(self.norms["norm"], self.norms["ffn_norm"], dt)
+        else:
+            x = x_ffn = stream.normed(self.norms["norm"], dt)
+        y = self.mixer.forward(x, ctx, cache)
+        if isinstance(y, Terms) or self.two_norms:
+            terms = list(y.pairs) if isinstance(y, Terms) else [(y, 1.0)]
+            if self.has_ffn:
+                terms.append((self.feed_forward.forward(x_ffn, ctx), 1.0))
+            stream.add_terms([(t, s * self.scale) for t, s in terms])
+            return
+        branches = [y]
         if self.has_ffn:
-            branches.append(self.feed_forward.forward(x, ctx))
+            branches.append(self.feed_forward.forward(x_ffn, ctx))
         stream.add_scaled(branches, self.scale)
 
 

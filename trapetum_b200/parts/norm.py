@@ -46,6 +46,17 @@ class RMSNorm(Norm):
         """``h += scale * (sum of the branch outputs)`` in place, returns ``norm(h)``; one kernel."""
         return ops.add_scaled_rmsnorm(h, branches, scale, self.weight, self.eps, self.offset, out_dtype)
 
+    def add_terms_apply(self, h: torch.Tensor, terms, out_dtype: torch.dtype, also: Optional["RMSNorm"] = None):
+        """``h += sum of scale * branch`` in place over (branch, scale) pairs; returns ``[norm(h)]``, or with ``also``
+        (another RMS norm of the same eps and form) ``[norm(h), also(h)]``; one kernel."""
+        return ops.add_terms_rmsnorm(h, terms, [self.weight] if also is None else [self.weight, also.weight], self.eps,
+                                     self.offset, out_dtype)
+
+    def shares_root(self, other) -> bool:
+        """Whether :meth:`add_terms_apply` takes ``other`` as its second norm."""
+        return isinstance(other, RMSNorm) and other.eps == self.eps and other.offset == self.offset \
+            and other.size == self.size and other.weight.dtype == self.weight.dtype
+
     def add_apply(self, h: torch.Tensor, a: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
         """``h += a`` in place (a branch output that no norm follows), returns ``norm(h)``; one kernel where the branch
         output is 32-bit (a matrix or split-K partial sums)."""

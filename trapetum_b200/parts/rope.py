@@ -8,6 +8,10 @@ is linear position scaling: every frequency is divided by f.  The table is made 
 32-bit; the kernel multiplies by the position and takes sin and cos in 32-bit.
 The rotation is fused with the cache write, so a mixer hands this part its qkv
 matrix and its cache line in one call.
+
+``pairing`` "neighbours" is the interleaved layout, pairs ``(x[2i], x[2i+1])``: a mixer that lays out its q and k
+heads in :meth:`Rope.head_order` (even places of the rotated part first) runs it as the rotate-half rotation.
+``table`` "float64" makes the frequencies in 64-bit before they are stored in 32.
 """
 from __future__ import annotations
 
@@ -63,7 +67,19 @@ class Rope(PositionEncoding):
         self._inv_freq_cpu = 1.0 / (torch.tensor(self.theta, dtype=torch.float32) ** (idx / self.rotary_dim))
         if self.scaling_factor != 1.0:
             self._inv_freq_cpu = self._inv_freq_cpu / self.scaling_factor
+        if params.get("table", "float32") == "float64":
+            self._inv_freq_cpu, _ = rotary_frequencies(self.rotary_dim, self.theta,
+                                                       {"factor": self.scaling_factor} if self.scaling_factor != 1.0 else None)
+        self.pairing = params.get("pairing", "halves")
+        if self.pairing not in ("halves", "neighbours"):
+            raise ValueError(f"rope: pairing '{self.pairing}' (known: halves, neighbours)")
         self.inv_freq: Optional[torch.Tensor] = None
+
+    def head_order(self):
+        if self.pairing == "halves":
+            return None
+        R = self.rotary_dim
+        return list(range(0, R, 2)) + list(range(1, R, 2)) + list(range(R, self.head_dim))
 
     def bind(self, tensors) -> None:
         self.inv_freq = self._inv_freq_cpu.to(self.rt.device)

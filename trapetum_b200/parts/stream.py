@@ -43,6 +43,11 @@ class ResidualStream:
         self._flush()
         self._pending = (list(branches), None, ("scaled", float(scale)))
 
+    def add_terms(self, terms) -> None:
+        """h += sum of scale * branch over up to three (branch output, scale) pairs, float32 or their split-K partial sums."""
+        self._flush()
+        self._pending = (list(terms), None, ("terms",))
+
     def fold_normed(self, a: torch.Tensor, norm: Norm, alpha: float) -> None:
         """h <- norm(alpha * h + a): the norm after the sum."""
         self._flush()
@@ -50,7 +55,11 @@ class ResidualStream:
 
     def normed(self, norm: Norm, out_dtype: torch.dtype) -> torch.Tensor:
         """norm(h), after whatever addition was still waiting."""
-        if self._pending is not None and isinstance(self._pending[2], tuple):
+        if self._pending is not None and self._pending[2] == ("terms",) and hasattr(norm, "add_terms_apply"):
+            terms = self._pending[0]
+            self._pending = None
+            return norm.add_terms_apply(self.h, terms, out_dtype)[0]      # the sum of the terms and the norm in one kernel
+        if self._pending is not None and isinstance(self._pending[2], tuple) and self._pending[2][0] == "scaled":
             branches, _, (_, scale) = self._pending
             if hasattr(norm, "add_scaled_apply"):
                 self._pending = None
@@ -65,6 +74,20 @@ class ResidualStream:
             ops.residual_add(self.h, a)
         self._flush()
         return norm.apply(self.h, out_dtype)
+
+    def normed_pair(self, first: Norm, second: Norm, out_dtype: torch.dtype):
+        """(first(h), second(h)), after whatever addition was still waiting: one kernel for a sum of terms (or none) and
+        two RMS norms of one form."""
+        terms = None
+        if self._pending is None:
+            terms = []
+        elif self._pending[2] == ("terms",):
+            terms = self._pending[0]
+        if terms is not None and hasattr(first, "add_terms_apply") and first.shares_root(second):
+            self._pending = None
+            a, b = first.add_terms_apply(self.h, terms, out_dtype, also=second)
+            return a, b
+        return self.normed(first, out_dtype), second.apply(self.h, out_dtype)
 
     def read(self, out_dtype: torch.dtype) -> torch.Tensor:
         """The stream itself for a sublayer that reads it unnormed: ``h`` when the compute dtype is 32-bit, else a
@@ -92,7 +115,9 @@ class ResidualStream:
             return
         a, post, alpha = self._pending
         self._pending = None
-        if isinstance(alpha, tuple):
+        if alpha == ("terms",):
+            ops.add_terms_rmsnorm(self.h, a)
+        elif isinstance(alpha, tuple):
             ops.add_scaled_rmsnorm(self.h, a, alpha[1])
         elif alpha is not None:
             post.fold(self.h, a, alpha, None)
