@@ -1496,17 +1496,26 @@ class _RetentionArgs(ctypes.Structure):
                 ("k_scale", c_float), ("eps", c_float), ("decay", c_void_p),
                 ("positions", c_void_p), ("token_seq", c_void_p), ("seq_start", c_void_p), ("slot_ids", c_void_p),
                 ("state", c_void_p), ("state_stride", c_longlong), ("rows", c_void_p), ("out", c_void_p),
-                ("batch", c_int), ("n_tokens", c_int)]
+                ("batch", c_int), ("n_tokens", c_int), ("chunk_sum", c_void_p), ("chunk_hi", c_void_p), ("chunk_lo", c_void_p),
+                ("chunk_len", c_int), ("n_chunks", c_int), ("row_blocks", c_int), ("DP", c_int), ("VP", c_int)]
+
+
+def retention_files(dtype: torch.dtype, key_dim: int, value_dim: int) -> Tuple[str, ...]:
+    """The kernel libraries that :func:`retention` launches for these sizes."""
+    lone = key_dim <= 256 and value_dim <= 512
+    return ("retention",) if lone and dtype == torch.bfloat16 else ("retention", "gla")
 
 
 def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_dtype: torch.dtype, rotary_dim: int,
               inv_freq: Optional[torch.Tensor], k_scale: float, decay: torch.Tensor, eps: float, state: torch.Tensor,
               positions: torch.Tensor, seq_start: torch.Tensor, token_seq: torch.Tensor, slot_ids: torch.Tensor, batch: int,
-              max_seq_len: int = 0) -> torch.Tensor:
+              max_seq_len: int = 0, generic: bool = False) -> torch.Tensor:
     """Retention between its products (see retention.cu).  ``part``: float32 partial sums [splits, T, >= 2 H D + 2 H V] of
     the input product, columns q, k, v and the gate; ``decay`` float32 [H]; ``state`` float32 [slots, H D V], rows picked
     by ``slot_ids``, read and written.  ``max_seq_len``: the longest sequence of a step of whole prompts, 0 for a step
-    of one token each.  Returns [T, H V] in ``out_dtype``."""
+    of one token each (which is then one launch, for ``key_dim`` up to 256 and ``value_dim`` up to 512).  Whole prompts run as
+    products over chunks in bfloat16 (the same sizes) and on the scan of gla.cu otherwise; ``generic``: the scan in any
+    case.  Returns [T, H V] in ``out_dtype``."""
     _cuda(part, inv_freq, decay, state, positions, seq_start, token_seq, slot_ids)
     HD, HV = heads * key_dim, heads * value_dim
     if part.dtype != torch.float32 or part.dim() != 3 or part.stride(2) != 1 or part.shape[2] < 2 * HD + 2 * HV:
@@ -1531,6 +1540,21 @@ def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_
     a.slot_ids = slot_ids.data_ptr(); a.state = state.data_ptr(); a.state_stride = state.stride(0)
     a.out = out.data_ptr(); a.batch = batch; a.n_tokens = T
     lib = build.load("retention")
+    if not generic and max_seq_len == 0 and T == batch and lib.tb_retention_step_takes(c_int(key_dim), c_int(value_dim)):
+        _check(lib, lib.tb_retention_step(ctypes.byref(a), c_int(code(out_dtype)), _stream()), "retention_step")
+        return out
+    if not generic and max_seq_len > 0 and lib.tb_retention_chunks_takes(c_int(code(out_dtype)), c_int(key_dim), c_int(value_dim)):
+        DP, VP = int(lib.tb_retention_padded_d(c_int(key_dim))), int(lib.tb_retention_padded_v(c_int(value_dim)))
+        C = int(lib.tb_retention_chunk_len(c_int(heads), c_int(value_dim), c_int(batch), c_int(int(max_seq_len)), c_int(sm_count(part.device))))
+        n_chunks, blocks = (max_seq_len + C - 1) // C, (max_seq_len + 127) // 128
+        if batch * blocks <= 65535:
+            rows = torch.empty((T, heads * (2 * DP + VP)), dtype=torch.bfloat16, device=part.device)
+            sums = torch.empty((batch, n_chunks, heads * DP * VP), dtype=torch.float32, device=part.device)
+            halves = torch.empty((2, batch, n_chunks, heads * DP * VP), dtype=torch.bfloat16, device=part.device)
+            a.rows = rows.data_ptr(); a.chunk_sum = sums.data_ptr(); a.chunk_hi = halves[0].data_ptr(); a.chunk_lo = halves[1].data_ptr()
+            a.chunk_len = C; a.n_chunks = n_chunks; a.row_blocks = blocks; a.DP = DP; a.VP = VP
+            _check(lib, lib.tb_retention_chunks(ctypes.byref(a), _stream()), "retention_chunks", 4)
+            return out
     rows = torch.empty((T, 2 * HD + 2 * HV), dtype=torch.float32, device=part.device)
     y = torch.empty((T, HV), dtype=torch.float32, device=part.device)
     a.rows = rows.data_ptr()

@@ -69,7 +69,7 @@ class Retention(Mixer):
         self.position.bind(tensors)
 
     def kernel_files(self):
-        return linear_kernels(self.rt.dtype) + ("retention", "gla")
+        return linear_kernels(self.rt.dtype) + ops.retention_files(self.rt.dtype, self.D, self.V)
 
     def cache_need(self):
         return StateNeed((self.heads * self.D * self.V,), torch.float32)
