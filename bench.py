@@ -22,6 +22,7 @@ MEASURED_PEAKS.json beside this file when the driver wrote it, otherwise from th
     python bench.py --design lofirax [--sizes small,medium,large] [--batch 8] [--context 2048]
     python bench.py --design fidepel [--sizes small,medium,large] [--batch 8] [--context 2048]
     python bench.py --design fibelix [--sizes small,medium,large] [--batch 8] [--context 2048]
+    python bench.py --design ranilix [--sizes small,medium,large] [--batch 8] [--context 2048]
 
 ``--design divanex`` is a measurement of its own (the default workload and its line stay as they are): Divanex
 models with random weights at a few layer sizes, a 2,048-token prompt and decode steps of ``batch`` sequences
@@ -1017,6 +1018,209 @@ def fibelix_compare(args, torch):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------------------
+# --design ranilix: the design at sizes that resemble real layers, beside Divanex (the closest model of the library:
+# attention layers and layers with a recurrent state in turn, dense feed-forwards, on the same host) at equal width, depth,
+# head counts, head size and vocabulary
+# ---------------------------------------------------------------------------------------------------------------
+# name -> (window; retention: heads, key size, value size); the rest are DESIGN_SIZES'
+RANILIX_SIZES = {"small": (1024, 8, 128, 256), "medium": (1024, 16, 128, 256), "large": (1024, 32, 128, 256)}
+
+
+def ranilix_config(size):
+    W, L, H, G, d, ff, _, _, _, V = DESIGN_SIZES[size]
+    win, rh, rd, rv = RANILIX_SIZES[size]
+    attn = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": win},
+                                           "rot": {"dims": d // 2, "base": 500000.0}, "v_mix": True}}
+    both = {"type": "parallel", "mixer": {
+        "left": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "rot": {"dims": d, "base": 10000.0}},
+        "right": {"heads": rh, "dim": rd, "vdim": rv, "rot": {"dims": rd, "base": 10000.0},
+                  "decay": [1.0 - 2.0 ** (-4 - 5.0 * i / rh) for i in range(rh)]},
+        "left_scale": 0.7, "right_scale": 0.6}}
+    for layer in (attn, both):
+        layer["mlp"] = {"kind": "dense", "ff": ff}
+    return {"architecture": "Ranilix", "vocab": V, "width": W, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "layers": [attn if i % 2 == 0 else both for i in range(L)]}
+
+
+def ranilix_bytes_flops(cfg, tokens, ctx, batch):
+    """(weight bytes a decode step reads, cache and state bytes per sequence at ``ctx`` tokens, tensor-core FLOPs of one
+    ``tokens``-token prompt with retention as the products over chunks of 128 tokens that its mathematics needs)."""
+    W, V = cfg["width"], cfg["vocab"]
+    wb, cb, fl = V * W + W, 0, 2 * V * W * tokens
+
+    def pairs(span):
+        span = min(tokens, span or tokens)
+        return span * (span + 1) // 2 + (tokens - span) * span
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        a = m["left"] if L["type"] == "parallel" else m
+        H, G, D, Vd = a["heads"], a["kv_heads"], a["dim"], a["vdim"]
+        size = (a.get("mask") or {}).get("size")
+        per = (H * D + G * (D + Vd)) * W + W * H * Vd + 2 * L["mlp"]["ff"] * W + 2 * W
+        cb += G * (D + Vd) * min(ctx, size or ctx) * 2
+        fl += 2 * H * (D + Vd) * pairs(size)
+        if L["type"] == "parallel":
+            r = m["right"]
+            h, D, Vd = r["heads"], r["dim"], r["vdim"]
+            per += h * (2 * D + 3 * Vd) * W
+            cb += 2 * 4 * h * D * Vd                                # the state is read and written, 32-bit
+            fl += h * tokens * (128 * (D + Vd) + 4 * D * Vd)
+        else:
+            per += H * Vd * W                                       # the gate
+        wb += per
+        fl += 2 * tokens * per
+    return 2 * wb, cb, fl, 0
+
+
+def ranilix_kernels(torch, size, hbm_gbs, tokens=PREFILL_TOKENS):
+    """The design's own kernels alone, each beside the like kernel of the library's other models: microseconds, algorithmic
+    bytes (or FLOPs) and the fraction of the roofline.  One prompt of ``tokens`` tokens; 64 sequences at 2,048 for the
+    one-token kernels."""
+    from trapetum_b200.csrc import ops
+    W, _, H, G, d, ff, mh, mp, N, _ = DESIGN_SIZES[size]
+    win, rh, rd, rv = RANILIX_SIZES[size]
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    T, B, ctx = tokens, 64, 2048
+    out = {}
+    tc_peak = peaks()[1]
+
+    def rec(name, us, nbytes, like=None, tensor_flops=0.0, fp32_flops=0.0):
+        t_mem, t_tc = nbytes / (hbm_gbs * 1e9) * 1e6, tensor_flops / (tc_peak * 1e12) * 1e6
+        t_fma = fp32_flops / (FP32_TFLOPS_NOMINAL * 1e12) * 1e6
+        best = max(t_mem, t_tc, t_fma)
+        out[name] = {"us": round(us, 1), "bytes": int(nbytes), "roofline_us": round(best, 1), "frac": round(best / us, 3),
+                     "bound": "tensor" if best == t_tc else ("fp32" if best == t_fma else "hbm")}
+        if like:
+            out[name]["like"] = like
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    rb = lambda *s: (torch.randn(*s, device=dev) * 0.5).to(bf)
+    pos, tseq = torch.arange(T, device=dev).int(), torch.zeros(T, device=dev).int()
+    ss, la = torch.tensor([0, T], device=dev).int(), torch.tensor([T], device=dev).int()
+    slot0 = torch.zeros(1, device=dev).int()
+    pos1 = torch.full((B,), ctx - 1, device=dev).int()
+    ss1, tseq1, la1 = torch.arange(B + 1, device=dev).int(), torch.arange(B, device=dev).int(), torch.full((B,), ctx, device=dev).int()
+    # ---- the sum of three branches with two norms, beside one branch with two norms
+    h, w1, w2 = f32(T, W), torch.ones(W, device=dev).to(bf), torch.ones(W, device=dev).to(bf)
+    br = [f32(1, T, W) for _ in range(3)]
+    rec("add_terms_rmsnorm (three branches, two norms)", _median_us(torch, lambda: ops.add_terms_rmsnorm(h, [(b, 0.7) for b in br], [w1, w2], 1e-6, 0.0, bf), flush),
+        T * W * (8 + 12 + 4), like="add_rmsnorm")
+    rec("add_rmsnorm", _median_us(torch, lambda: ops.add_rmsnorm(h, br[0], w1, 1e-5, 0.0, w2, 1e-5, 0.0, bf), flush), T * W * 14)
+    # ---- between the attention's products and its kernel
+    pages = (T + 63) // 64
+    inv = torch.rand(d // 4, device=dev)
+    wide = (H * d + 2 * G * d + H * d + 15) // 16 * 16
+    bias = f32(wide)
+    wn, wq, wk = torch.ones(d, device=dev), torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+    ones = torch.ones(H, device=dev)
+    for what, TT, po, ts, le, splits in (("", T, pos, tseq, la, 1), (", one token for each of 64 sequences", B, pos1, tseq1, la1, 4)):
+        part, part0 = f32(splits, TT, wide), f32(splits, TT, (H * d + 2 * G * d + H + 15) // 16 * 16)
+        first = f32(TT, G * d)
+        n_seq = le.numel()
+        kp, vp = (torch.zeros(n_seq * pages, G, 64, d, dtype=bf, device=dev) for _ in range(2))
+        table = torch.arange(n_seq * pages, device=dev).int().view(n_seq, pages)
+        nb = TT * (H + 2 * G) * d * (4 * splits + 2) + TT * 2 * G * d * 2
+        rec("projnorm_kv (head norms, biases, mixed values)" + what,
+            _median_us(torch, lambda: ops.projnorm_kv(part, H, G, d, d, d, bf, wn, wn, 1e-6, None, d // 2, inv, False, po, ts, le, kp, vp, table, 0,
+                                                      bias, True, first, 0.3), flush),
+            nb + TT * G * d * 4, like="projnorm_kv (norms over the projection)" + what)
+        rec("projnorm_kv (norms over the projection)" + what,
+            _median_us(torch, lambda: ops.projnorm_kv(part0, H, G, d, d, d, bf, wq, wk, 1e-6, ones, d // 2, inv, True, po, ts, le, kp, vp, table, 0), flush), nb)
+        o, gate = rb(TT, H * d), torch.rand(TT, H, device=dev)
+        rec("value_gate" + what, _median_us(torch, lambda: ops.value_gate(o, part[:, :, H * d + 2 * G * d:H * d + 2 * G * d + H * d], H, d), flush),
+            TT * H * d * (4 * splits + 4), like="head_gate" + what)
+        rec("head_gate" + what, _median_us(torch, lambda: ops.head_gate(o, gate, H), flush), TT * H * d * 4)
+    # ---- attention with a sink and a window, beside the same kernel without a sink
+    q, k, v, sink = rb(T, H * d), rb(T, G * d), rb(T, G * d), torch.ones(H, device=dev)
+    n_pairs = win * (win + 1) // 2 + (T - win) * win
+    nb = (2 * H + 2 * G) * d * T * 2
+    rec("attention with a sink (prefill)", _median_us(torch, lambda: ops.attn_prefill_sink(q, k, v, ss, tseq, H, d, d ** -0.5, sink, T, [T], win, n_kv_heads=G), flush),
+        nb, like="attention (prefill)", tensor_flops=4.0 * H * d * n_pairs)
+    rec("attention (prefill)", _median_us(torch, lambda: ops.attn_prefill(q, k, v, ss, tseq, H, G, d, d ** -0.5, 0.0, win, T, [T]), flush),
+        nb, tensor_flops=4.0 * H * d * n_pairs)
+    ring = win
+    kp, vp = rb(B * ring // 64, G, 64, d), rb(B * ring // 64, G, 64, d)
+    tab, q1 = torch.arange(B * ring // 64, device=dev).int().view(B, ring // 64), rb(B, H * d)
+    for name, s in (("attention with a sink (decode)", sink), ("attention (decode)", None)):
+        rec(name, _median_us(torch, lambda: ops.attn_decode(q1, kp, vp, tab, la1, H, G, d, d ** -0.5, 0.0, win, ring, ctx, sink=s), flush),
+            B * 2 * G * d * win * 2, like="attention (decode)" if s is not None else None)
+    # ---- retention, beside gated linear attention (a decay per key channel) and the state-space mixer
+    HD, HV = rh * rd, rh * rv
+    rinv, dec = torch.rand(rd // 2, device=dev), torch.full((rh,), 0.99, device=dev)
+    low, a2, a2b, nw = f32(1, T, 16), f32(HD, 16) * .3, f32(HD) + 2, torch.ones(rv, device=dev)
+    st, st64 = torch.zeros(1, HD * rv, device=dev), torch.zeros(B, HD * rv, device=dev)
+    part = f32(1, T, 2 * HD + 2 * HV)
+    nb = T * ((2 * HD + 2 * HV) * 4 + HV * 2)
+    rec("retention (prompt)", _median_us(torch, lambda: ops.retention(part, rh, rd, rv, bf, rd, rinv, rd ** -0.5, dec, 1e-6, st, pos, ss, tseq, slot0, 1, T), flush),
+        nb, like="gla (prompt)", tensor_flops=rh * T * (128.0 * (rd + rv) + 4.0 * rd * rv))
+    proj = rb(T, 2 * HD + 2 * HV)
+    rec("gla (prompt)", _median_us(torch, lambda: ops.gla(proj, low, a2, a2b, 8.0, rd ** -0.5, nw, 1e-6, rh, rd, rv, st, ss, tseq, slot0, 1, max_seq_len=T), flush),
+        T * ((2 * HD + 2 * HV) * 2 + HD * 4 * 2 + HV * 4 * 2 + HV * 2), fp32_flops=T * HD * rv * 5.0)
+    part1, proj1, low1 = f32(4, B, 2 * HD + 2 * HV), rb(B, 2 * HD + 2 * HV), f32(1, B, 16)
+    rec("retention, one token for each of 64 sequences",
+        _median_us(torch, lambda: ops.retention(part1, rh, rd, rv, bf, rd, rinv, rd ** -0.5, dec, 1e-6, st64, pos1, ss1, tseq1, tseq1, B), flush),
+        st64.numel() * 8 + part1.numel() * 4, like="gla, one token for each of 64 sequences")
+    rec("gla, one token for each of 64 sequences",
+        _median_us(torch, lambda: ops.gla(proj1, low1, a2, a2b, 8.0, rd ** -0.5, nw, 1e-6, rh, rd, rv, st64, ss1, tseq1, tseq1, B), flush), st64.numel() * 8)
+    inner, ch = mh * mp, mh * mp + 2 * N
+    mproj1, dtr1 = rb(B, inner + ch), f32(B, mh)
+    cw, cb_, dtb, Al, Dm, mnw = f32(ch, 4) * .3, f32(ch) * .1, f32(mh) - 1, f32(mh) * .5, f32(mh), f32(inner)
+    ms = torch.zeros(B, ops.mamba2_state_size(mh, mp, N, 1, 4), device=dev)
+    rec("mamba2, one token for each of 64 sequences",
+        _median_us(torch, lambda: ops.mamba2(mproj1, dtr1, mh, mp, N, 1, 4, 1, cw, cb_, dtb, Al, Dm, mnw, 1e-5, ms, ss1, tseq1, tseq1, B, True), flush), ms.numel() * 8)
+    return out
+
+
+def ranilix_compare(args, torch):
+    """Prints one JSON line: per size, Ranilix and the Divanex model of equal width, depth, heads and vocabulary (prefill of
+    one 2,048-token prompt, decode at ``batch`` x ``context``), with bytes, FLOPs and roofline fractions, and the design's
+    kernels alone beside their like kernels."""
+    import trapetum_b200 as tb
+    from trapetum_b200.csrc import ops
+    hbm_gbs, bf16_tflops, peak_src = peaks()
+    warmup = max(3, args.warmup)
+    ctx, batch = args.context, args.batch
+    out = {"design": "ranilix", "beside": "divanex", "sizes": {},
+           "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": bf16_tflops, "source": peak_src, "fp32_tflops_nominal": FP32_TFLOPS_NOMINAL},
+           "dtype": "bf16", "data": "synthetic (random weights, random token ids)", "batch": batch, "context": ctx,
+           "timing": "CUDA events; decode: median of five regions of --steps steps; kernels alone: a 256 MB buffer is written "
+                     "between timed launches (larger than L2)"}
+    clocks = ClockSampler()
+    clocks.__enter__()
+    for size in [s for s in args.sizes.split(",") if s in DESIGN_SIZES]:
+        row = {}
+        for which in ("ranilix", "divanex"):
+            cfg = ranilix_config(size) if which == "ranilix" else divanex_config(size)
+            V = cfg["vocab"]
+            model = tb.random_model(cfg, 7, 0.02, 0.1, "bfloat16", "cuda:0", host="python")
+            engine = tb.Engine(model, max_tokens=batch * (ctx + 64), max_slots=batch)
+            random_cache(engine)
+            pms, _, _ = time_prefill(engine, torch, PREFILL_TOKENS, V, reps=5, warmup=warmup)
+            r = time_decode(engine, torch, [ctx] * batch, args.steps, warmup, V, clocks=clocks)
+            wb, cb, fl, rf = (ranilix_bytes_flops if which == "ranilix" else divanex_bytes_flops)(cfg, PREFILL_TOKENS, ctx, batch)
+            nbytes = wb + batch * cb
+            pre_ideal = fl / (bf16_tflops * 1e12) + rf / (FP32_TFLOPS_NOMINAL * 1e12)
+            row[which] = {
+                "prefill": {"tokens": PREFILL_TOKENS, "ms": round(pms, 3), "tok_s": round(PREFILL_TOKENS * 1e3 / pms, 1),
+                            "tensor_flops": fl, "fp32_recurrence_flops": rf, "frac_of_roofline": round(pre_ideal * 1e3 / pms, 4)},
+                "decode": {"ms": r["ms"], "tok_s": round(batch * 1e3 / r["ms"], 1), "bytes": nbytes,
+                           "gbs": round(nbytes / (r["ms"] * 1e-3) / 1e9, 1),
+                           "frac_of_hbm": round(nbytes / (r["ms"] * 1e-3) / 1e9 / hbm_gbs, 4), "launches": r["launches"]},
+            }
+            engine.check_kernels()
+            del engine, model
+            torch.cuda.empty_cache()
+        if not args.no_points:
+            row["kernels_alone"] = ranilix_kernels(torch, size, hbm_gbs)
+        out["sizes"][size] = row
+    clocks.__exit__()
+    out["clocks"] = clocks.summary()
+    out["kernel_errors"] = ops.kernel_errors()
+    print(json.dumps(out))
+    return 0
+
+
 HOST = None              # which host runs the models (None: the library's default, the native host for these models)
 
 
@@ -1365,7 +1569,7 @@ def main() -> int:
     ap.add_argument("--leave-out", action="store_true",
                     help="instead of the bench line: the decode step re-timed with one kind of launch left out at a "
                          "time (its results are then wrong; only its time is of interest), one line per kind")
-    ap.add_argument("--design", default=None, choices=["divanex", "lofirax", "fidepel", "fibelix"],
+    ap.add_argument("--design", default=None, choices=["divanex", "lofirax", "fidepel", "fibelix", "ranilix"],
                     help="instead of the bench line: this design at the layer sizes of --sizes beside the library's closest "
                          "model at equal size (divanex beside Gemma-2, lofirax beside divanex, fidepel beside Gemma-2, fibelix beside fidepel)")
     ap.add_argument("--sizes", default="small,medium,large", help="with --design: which of small, medium, large")
@@ -1393,6 +1597,8 @@ def main() -> int:
             return fidepel_compare(args, torch)
         if args.design == "fibelix":
             return fibelix_compare(args, torch)
+        if args.design == "ranilix":
+            return ranilix_compare(args, torch)
         return lofirax_compare(args, torch) if args.design == "lofirax" else design_compare(args, torch)
     if args.gemm_compare:
         return gemm_compare(MODELS[args.model], torch, args.gemm_compare, peaks()[1])
