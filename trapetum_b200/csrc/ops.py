@@ -1502,7 +1502,7 @@ class _RetentionArgs(ctypes.Structure):
 
 def retention_files(dtype: torch.dtype, key_dim: int, value_dim: int) -> Tuple[str, ...]:
     """The kernel libraries that :func:`retention` launches for these sizes."""
-    lone = key_dim <= 256 and value_dim <= 512
+    lone = key_dim <= 256 and value_dim <= 512 and value_dim % 4 == 0
     return ("retention",) if lone and dtype == torch.bfloat16 else ("retention", "gla")
 
 
@@ -1513,8 +1513,8 @@ def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_
     """Retention between its products (see retention.cu).  ``part``: float32 partial sums [splits, T, >= 2 H D + 2 H V] of
     the input product, columns q, k, v and the gate; ``decay`` float32 [H]; ``state`` float32 [slots, H D V], rows picked
     by ``slot_ids``, read and written.  ``max_seq_len``: the longest sequence of a step of whole prompts, 0 for a step
-    of one token each (which is then one launch, for ``key_dim`` up to 256 and ``value_dim`` up to 512).  Whole prompts run as
-    products over chunks in bfloat16 (the same sizes) and on the scan of gla.cu otherwise; ``generic``: the scan in any
+    of one token each (which is then one launch, for ``value_dim`` up to 512 in multiples of 4).  Whole prompts run as
+    products over chunks in bfloat16 (``key_dim`` up to 256, ``value_dim`` up to 512) and on the scan of gla.cu otherwise; ``generic``: the scan in any
     case.  Returns [T, H V] in ``out_dtype``."""
     _cuda(part, inv_freq, decay, state, positions, seq_start, token_seq, slot_ids)
     HD, HV = heads * key_dim, heads * value_dim
@@ -1540,8 +1540,8 @@ def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_
     a.slot_ids = slot_ids.data_ptr(); a.state = state.data_ptr(); a.state_stride = state.stride(0)
     a.out = out.data_ptr(); a.batch = batch; a.n_tokens = T
     lib = build.load("retention")
-    if not generic and max_seq_len == 0 and T == batch and lib.tb_retention_step_takes(c_int(key_dim), c_int(value_dim)):
-        _check(lib, lib.tb_retention_step(ctypes.byref(a), c_int(code(out_dtype)), _stream()), "retention_step")
+    if not generic and max_seq_len == 0 and T == batch and state.data_ptr() % 16 == 0 and state.stride(0) % 4 == 0 and lib.tb_retention_step_takes(c_int(key_dim), c_int(value_dim)):
+        _check(lib, lib.tb_retention_step(ctypes.byref(a), c_int(code(out_dtype)), c_int(sm_count(part.device)), _stream()), "retention_step")
         return out
     if not generic and max_seq_len > 0 and lib.tb_retention_chunks_takes(c_int(code(out_dtype)), c_int(key_dim), c_int(value_dim)):
         DP, VP = int(lib.tb_retention_padded_d(c_int(key_dim))), int(lib.tb_retention_padded_v(c_int(value_dim)))

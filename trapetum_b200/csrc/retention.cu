@@ -6,17 +6,17 @@
 // head's o_t is then divided by its root mean square over v and multiplied by silu(g_t).  The input is the product as
 // 32-bit partial sums; a sequence's state is a 32-bit row addressed by slot.
 //
-//   tb_retention_step   one token per sequence: everything in one launch.  A cluster of CTAs owns one head of one
-//                       sequence, each CTA 64 value channels with all key channels of them in registers (fetched while
-//                       the product before is still running); the CTAs exchange their sums of squares through
-//                       distributed shared memory.
+//   tb_retention_step   one token per sequence: everything in one launch.  A CTA owns one head of one sequence and
+//                       streams its state through registers; the first rows are fetched while the product before is
+//                       still running.
 //   tb_retention_chunks whole prompts in bfloat16, as matrix products over chunks of C tokens (mma.sync): with i, j
 //                       places in a chunk and S the state before it,
 //                           o_i = sum_{j <= i} decay^(i - j) (q_i . k_j) v_j + decay^(i + 1) S^T q_i
 //                           S'  = decay^n S + sum_j decay^(n - 1 - j) k_j v_j^T           (n tokens in the chunk)
 //                       in four launches: rows prepared (turned, scaled, padded, rounded once), each chunk's own sum E,
 //                       the states before the chunks from the E (a scan over chunks, element by element), and the outputs
-//                       with norm and gate (again a cluster of CTAs per head, 64 value channels each).
+//                       with norm and gate (a cluster of CTAs owns a head, each of them 64 value channels; they
+//                       exchange their sums of squares through distributed shared memory).
 //   tb_retention_prep   the 32-bit rows [q | k | v | g] for the scan of gla.cu (any sizes, both dtypes)
 //
 // 32-bit: angles, rotation, decays, the state, o, its norm and the gate.  v is a product's output and is rounded to the
@@ -108,100 +108,123 @@ __global__ void __launch_bounds__(256) retention_prep_kernel(RetentionArgs a) {
 // ---------------------------------------------------------------------------
 // One token per sequence
 // ---------------------------------------------------------------------------
-constexpr int STEP_WARPS = 8;
+// A lane owns NC groups of four neighbouring value channels; LPR lanes (16 or 32) span a row of the state, so a warp
+// takes 32 / LPR key channels at a time, with 16-byte loads and stores.
 
-template <typename T, int DPT>
-__global__ void __launch_bounds__(STEP_WARPS * 32) retention_step_kernel(RetentionArgs a) {
+template <typename T, int NC, int LPR>
+__global__ void __launch_bounds__(1024) retention_step_kernel(RetentionArgs a) {
     pdl_launch_dependents();
-    constexpr int DMAX = DPT * STEP_WARPS;
-    __shared__ float raw_s[2][DMAX], q_s[DMAX], k_s[DMAX], cs[DMAX / 2 + 1], sn[DMAX / 2 + 1];
-    __shared__ float v_s[VT], g_s[VT], part_s[STEP_WARPS][VT], ss_s[2], total_s;
-    cg::cluster_group cluster = cg::this_cluster();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * VT;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[33];
+    constexpr int RPW = 32 / LPR;                     // rows of the state per pass of a warp
+    constexpr int STEP_ROWS = NC > 2 ? 2 : 4;         // passes whose loads are in flight together
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarp = blockDim.x >> 5;
+    const int h = blockIdx.x, b = blockIdx.y;
     const int D = a.D, V = a.V, HD = a.heads * D, HV = a.heads * V, half = a.rotary_dim >> 1;
+    float* raw_s = sm;                                // [2 D] q, k as the product left them
+    float* q_s = raw_s + 2 * D;                       // [D]
+    float* k_s = q_s + D;                             // [D]
+    float* cs = k_s + D;                              // [D / 2 rounded up] each
+    float* sn = cs + (D + 1) / 2;
+    float* v_s = sm + (((5 * D + 2) + 3) & ~3);       // [V], 16-byte aligned
+    float* g_s = v_s + V;                             // [V]
+    float* part_s = g_s + V;                          // [nwarp][V]
+    const int sub = lane % LPR, r_in = lane / LPR;
     // The step's integer inputs were copied before its first kernel, and this sequence's state was last written in an
     // earlier step (or zeroed when its slot was claimed): both may be read ahead of the wait.
     float* st = a.state + (size_t)a.slot_ids[b] * a.state_stride + (size_t)h * D * V;
-    const int vc[2] = {v0 + lane, v0 + lane + 32};
-    const bool v_ok[2] = {vc[0] < V, vc[1] < V};
-    float S[2][DPT];
+    const int passes = (D + nwarp * RPW - 1) / (nwarp * RPW);
+    float4 S[STEP_ROWS][NC];
+    auto row_of = [&](int p) { return (p * nwarp + warp) * RPW + r_in; };
+    auto fetch = [&](int p0) {
 #pragma unroll
-    for (int j = 0; j < DPT; j++) {
-        const int d = warp * DPT + j;
+        for (int u = 0; u < STEP_ROWS; u++) {
+            const int d = row_of(p0 + u);
 #pragma unroll
-        for (int c = 0; c < 2; c++) S[c][j] = (d < D && v_ok[c]) ? st[(size_t)d * V + vc[c]] : 0.f;
-    }
+            for (int c = 0; c < NC; c++) {
+                const int v = (c * LPR + sub) * 4;
+                S[u][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (p0 + u < passes && d < D && v < V) S[u][c] = *(const float4*)(st + (size_t)d * V + v);
+            }
+        }
+    };
+    fetch(0);
     const float dec = a.decay[h];
     const int pos = a.positions[b];
     for (int i = tid; i < half; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &sn[i], &cs[i]);
     pdl_wait();
     const float* src = a.part + (size_t)b * a.row_stride;
-    for (int u = tid; u < 2 * D + 2 * VT; u += blockDim.x) {
-        int c = -1;
-        if (u < D) c = h * D + u;
-        else if (u < 2 * D) c = HD + h * D + (u - D);
-        else if (u < 2 * D + VT) { if (v0 + (u - 2 * D) < V) c = 2 * HD + h * V + v0 + (u - 2 * D); }
-        else if (v0 + (u - 2 * D - VT) < V) c = 2 * HD + HV + h * V + v0 + (u - 2 * D - VT);
-        float s = 0.f;
-        if (c >= 0) {
-            s = src[c];
+    for (int u = tid; u < 2 * D + 2 * V; u += blockDim.x) {
+        const int c = u < D ? h * D + u : u < 2 * D ? HD + h * D + (u - D) : u < 2 * D + V ? 2 * HD + h * V + (u - 2 * D)
+                                                                                            : 2 * HD + HV + h * V + (u - 2 * D - V);
+        float s = src[c];
 #pragma unroll 8
-            for (int sp = 1; sp < a.n_splits; sp++) s += src[(size_t)sp * a.split_stride + c];
-        }
-        if (u < D) raw_s[0][u] = s;
-        else if (u < 2 * D) raw_s[1][u - D] = s;
-        else if (u < 2 * D + VT) v_s[u - 2 * D] = kept<T>(s);
-        else g_s[u - 2 * D - VT] = s;
+        for (int sp = 1; sp < a.n_splits; sp++) s += src[(size_t)sp * a.split_stride + c];
+        if (u < 2 * D) raw_s[u] = s;
+        else if (u < 2 * D + V) v_s[u - 2 * D] = kept<T>(s);
+        else g_s[u - 2 * D - V] = s;
     }
     __syncthreads();
-    for (int u = tid; u < 2 * DMAX; u += blockDim.x) {
-        const int w = u >= DMAX, i = u - w * DMAX;
-        const float* x = raw_s[w];
-        float y = 0.f;
-        if (i < half) y = x[i] * cs[i] - x[i + half] * sn[i];
-        else if (i < 2 * half) y = x[i] * cs[i - half] + x[i - half] * sn[i - half];
-        else if (i < D) y = x[i];
+    for (int u = tid; u < 2 * D; u += blockDim.x) {
+        const int w = u >= D, i = u - w * D;
+        const float* x = raw_s + w * D;
+        const float y = i < half ? x[i] * cs[i] - x[i + half] * sn[i]
+                      : i < 2 * half ? x[i] * cs[i - half] + x[i - half] * sn[i - half] : x[i];
         if (w) k_s[i] = y * a.k_scale; else q_s[i] = y;
     }
     __syncthreads();
-    const float va = v_s[lane], vb = v_s[lane + 32];
-    float acc_a = 0.f, acc_b = 0.f;
+    float4 acc[NC];
 #pragma unroll
-    for (int j = 0; j < DPT; j++) {
-        const int d = warp * DPT + j;
-        const float kk = k_s[d], qq = q_s[d];
-        S[0][j] = fmaf(dec, S[0][j], kk * va);
-        S[1][j] = fmaf(dec, S[1][j], kk * vb);
-        acc_a = fmaf(S[0][j], qq, acc_a);
-        acc_b = fmaf(S[1][j], qq, acc_b);
+    for (int c = 0; c < NC; c++) acc[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int p0 = 0; p0 < passes; p0 += STEP_ROWS) {
+        if (p0 > 0) fetch(p0);
+#pragma unroll
+        for (int u = 0; u < STEP_ROWS; u++) {
+            const int d = row_of(p0 + u);
+            const bool in = p0 + u < passes && d < D;
+            const float kk = in ? k_s[d] : 0.f, qq = in ? q_s[d] : 0.f;
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                const int v = (c * LPR + sub) * 4;
+                if (!in || v >= V) continue;
+                const float4 x = *(const float4*)(v_s + v);
+                float4& s = S[u][c];
+                s.x = fmaf(dec, s.x, kk * x.x); s.y = fmaf(dec, s.y, kk * x.y);
+                s.z = fmaf(dec, s.z, kk * x.z); s.w = fmaf(dec, s.w, kk * x.w);
+                acc[c].x = fmaf(s.x, qq, acc[c].x); acc[c].y = fmaf(s.y, qq, acc[c].y);
+                acc[c].z = fmaf(s.z, qq, acc[c].z); acc[c].w = fmaf(s.w, qq, acc[c].w);
+                *(float4*)(st + (size_t)d * V + v) = s;
+            }
+        }
     }
-    part_s[warp][lane] = acc_a;
-    part_s[warp][lane + 32] = acc_b;
+    if (LPR == 16) {                                  // the two rows of a pass meet
 #pragma unroll
-    for (int j = 0; j < DPT; j++) {
-        const int d = warp * DPT + j;
+        for (int c = 0; c < NC; c++) {
+            acc[c].x += __shfl_xor_sync(0xffffffffu, acc[c].x, 16); acc[c].y += __shfl_xor_sync(0xffffffffu, acc[c].y, 16);
+            acc[c].z += __shfl_xor_sync(0xffffffffu, acc[c].z, 16); acc[c].w += __shfl_xor_sync(0xffffffffu, acc[c].w, 16);
+        }
+    }
 #pragma unroll
-        for (int c = 0; c < 2; c++) if (d < D && v_ok[c]) st[(size_t)d * V + vc[c]] = S[c][j];
+    for (int c = 0; c < NC; c++) {
+        const int v = (c * LPR + sub) * 4;
+        if (r_in == 0 && v < V) *(float4*)(part_s + (size_t)warp * V + v) = acc[c];
     }
     __syncthreads();
-    float o = 0.f;
-    if (tid < VT) {
+    // a thread sums up to two channels (V is at most twice the smallest block)
+    float o[2] = {0.f, 0.f};
 #pragma unroll
-        for (int w = 0; w < STEP_WARPS; w++) o += part_s[w][tid];
-        const float q2 = warp_sum(o * o);             // channels past V hold zeros
-        if (lane == 0) ss_s[warp] = q2;
+    for (int e = 0; e < 2; e++) {
+        const int v = tid + e * blockDim.x;
+        if (v < V) for (int w = 0; w < nwarp; w++) o[e] += part_s[(size_t)w * V + v];
     }
-    __syncthreads();
-    if (tid == 0) total_s = ss_s[0] + ss_s[1];
-    cluster.sync();
-    float ss = 0.f;
-    for (unsigned r = 0; r < cluster.num_blocks(); r++) ss += *cluster.map_shared_rank(&total_s, r);
-    cluster.sync();                                   // nobody leaves while its sum may still be read
-    if (tid < VT && v0 + tid < V) {
-        const float r = 1.f / sqrtf(ss / (float)V + a.eps);
-        const float g = g_s[tid];
-        ((T*)a.out)[(size_t)b * HV + (size_t)h * V + v0 + tid] = from_f<T>(o * r * (g / (1.f + expf(-g))));
+    const float ss = block_sum(o[0] * o[0] + o[1] * o[1], red);
+    const float r = 1.f / sqrtf(ss / (float)V + a.eps);
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+        const int v = tid + e * blockDim.x;
+        if (v >= V) continue;
+        const float g = g_s[v];
+        ((T*)a.out)[(size_t)b * HV + (size_t)h * V + v] = from_f<T>(o[e] * r * (g / (1.f + expf(-g))));
     }
 }
 
@@ -576,6 +599,28 @@ __global__ void __launch_bounds__(CT) retention_out_kernel(RetentionArgs a) {
         }
         __syncthreads();
     }
+    // ---- the gate's columns, on their way while the CTAs exchange their sums
+    const int HD = a.heads * a.D, HV = a.heads * a.V;
+    const bool pairs = a.n_splits == 1 && (a.V & 1) == 0 && (a.row_stride & 1) == 0 && ((uintptr_t)a.part & 7) == 0;
+    float2 gv[2][8];
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+        const int row = r0 + warp * 16 + g + e * 8;
+        const float* gp = a.part + (size_t)(s0 + min(row, len - 1)) * a.row_stride + 2 * HD + HV + (size_t)h * a.V;
+#pragma unroll
+        for (int j = 0; j < 8; j++) {
+            const int c = blockIdx.x * VT + j * 8 + 2 * t;
+            gv[e][j] = make_float2(0.f, 0.f);
+            if (pairs) {
+                if (c < a.V) gv[e][j] = __ldg((const float2*)(gp + c));
+            } else {
+                for (int sp = 0; sp < a.n_splits; sp++) {
+                    if (c < a.V) gv[e][j].x += gp[(size_t)sp * a.split_stride + c];
+                    if (c + 1 < a.V) gv[e][j].y += gp[(size_t)sp * a.split_stride + c + 1];
+                }
+            }
+        }
+    }
     // ---- the head's root mean square over all its CTAs, the gate, the store
     float sa = 0.f, sb = 0.f;
 #pragma unroll
@@ -590,26 +635,19 @@ __global__ void __launch_bounds__(CT) retention_out_kernel(RetentionArgs a) {
         ra += peer[warp * 16 + g]; rbs += peer[warp * 16 + g + 8];
     }
     cluster.sync();                                   // nobody leaves while its sums may still be read
-    const int HD = a.heads * a.D, HV = a.heads * a.V;
 #pragma unroll
     for (int e = 0; e < 2; e++) {
         const int row = r0 + warp * 16 + g + e * 8;
         if (row >= len) continue;
         const float r = 1.f / sqrtf((e ? rbs : ra) / (float)a.V + a.eps);
-        const float* gp = a.part + (size_t)(s0 + row) * a.row_stride + 2 * HD + HV + (size_t)h * a.V;
         bf16* op = (bf16*)a.out + (size_t)(s0 + row) * HV + (size_t)h * a.V;
 #pragma unroll
         for (int j = 0; j < 8; j++) {
             const int c = blockIdx.x * VT + j * 8 + 2 * t;
-            float y[2];
-#pragma unroll
-            for (int k = 0; k < 2; k++) {
-                float gv = 0.f;
-                if (c + k < a.V) for (int sp = 0; sp < a.n_splits; sp++) gv += gp[(size_t)sp * a.split_stride + c + k];
-                y[k] = o[j][e * 2 + k] * r * (gv / (1.f + __expf(-gv)));
-            }
-            if (c + 1 < a.V && (a.V & 1) == 0) *(uint32_t*)(op + c) = pack_bf16(y[0], y[1]);
-            else { if (c < a.V) op[c] = __float2bfloat16_rn(y[0]); if (c + 1 < a.V) op[c + 1] = __float2bfloat16_rn(y[1]); }
+            const float y0 = o[j][e * 2] * r * (gv[e][j].x / (1.f + __expf(-gv[e][j].x)));
+            const float y1 = o[j][e * 2 + 1] * r * (gv[e][j].y / (1.f + __expf(-gv[e][j].y)));
+            if ((a.V & 1) == 0) { if (c < a.V) *(uint32_t*)(op + c) = pack_bf16(y0, y1); }
+            else { if (c < a.V) op[c] = __float2bfloat16_rn(y0); if (c + 1 < a.V) op[c + 1] = __float2bfloat16_rn(y1); }
         }
     }
 }
@@ -633,26 +671,28 @@ extern "C" int tb_retention_prep(const RetentionArgs* args, int dtype, cudaStrea
     return tb_launch_status();
 }
 
-// Whether one launch takes a step of one token per sequence: a head's value channels fit a cluster of eight CTAs.
-extern "C" int tb_retention_step_takes(int D, int V) { return D >= 1 && D <= 256 && V >= 1 && V <= 8 * VT; }
+// Whether one launch takes a step of one token per sequence.
+extern "C" int tb_retention_step_takes(int D, int V) { return D >= 1 && D <= 1024 && V >= 4 && V <= 512 && V % 4 == 0; }
 
-extern "C" int tb_retention_step(const RetentionArgs* args, int dtype, cudaStream_t stream) {
+extern "C" int tb_retention_step(const RetentionArgs* args, int dtype, int sms, cudaStream_t stream) {
     const RetentionArgs& a = *args;
     if (a.batch <= 0) return 0;
     if (check(a)) return -1;
-    if (!tb_retention_step_takes(a.D, a.V)) return tb_refuse("retention: the one-token kernel takes D up to 256 and V up to 512, got %d and %d", a.D, a.V);
+    if (!tb_retention_step_takes(a.D, a.V))
+        return tb_refuse("retention: the one-token kernel takes D up to 1024 and V up to 512 in multiples of 4, got %d and %d", a.D, a.V);
     if (a.n_tokens != a.batch) return tb_refuse("retention: %d tokens for %d sequences in a step of one token each", a.n_tokens, a.batch);
-    const int nv = (a.V + VT - 1) / VT;
-    const dim3 grid(nv, a.heads, a.batch);
-    int dpt = 4;
-    while (dpt * STEP_WARPS < a.D) dpt <<= 1;
-#define RSTEP(N) TB_DISPATCH_1(dtype, T, launch_cluster(retention_step_kernel<T, N>, grid, dim3(STEP_WARPS * 32), 0, nv, stream, a))
-    switch (dpt) {
-    case 4: RSTEP(4); break;
-    case 8: RSTEP(8); break;
-    case 16: RSTEP(16); break;
-    default: RSTEP(32); break;
-    }
+    if (((uintptr_t)a.state & 15) || a.state_stride % 4) return tb_refuse("retention: states must be 16-byte aligned");
+    // few (head, sequence) pairs: more threads for each, so that a state's rows are all in flight at once
+    const long long ctas = (long long)a.heads * a.batch;
+    const int threads = ctas <= sms ? 1024 : ctas <= 2LL * sms ? 512 : 256;
+    const size_t smem = (size_t)((((5 * a.D + 2) + 3) & ~3) + 2 * a.V + (threads / 32) * a.V) * sizeof(float);
+#define RSTEP(NC, LPR) do { \
+        if (smem > 48 * 1024) { \
+            cudaError_t e = cudaFuncSetAttribute(retention_step_kernel<T, NC, LPR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024); \
+            if (e != cudaSuccess) return (int)e; \
+        } \
+        tb_launch(retention_step_kernel<T, NC, LPR>, dim3(a.heads, a.batch), dim3(threads), smem, stream, a); } while (0)
+    TB_DISPATCH_1(dtype, T, if (a.V <= 64) RSTEP(1, 16); else if (a.V <= 128) RSTEP(1, 32); else if (a.V <= 256) RSTEP(2, 32); else RSTEP(4, 32));
 #undef RSTEP
     return tb_launch_status();
 }
