@@ -296,6 +296,35 @@ def test_retention_between_its_products(H, D, V, R, decay, dtype, generic):
                 assert torch.equal(state[s], untouched[s])
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("decay", [0.9, 0.0])
+def test_a_tokens_own_product_keeps_its_sign(dtype, decay):
+    """A sequence's first token (and every token of a head that forgets at once) gives (q . k) v, of which the norm leaves
+    the sign of q . k: products that nearly cancel, in a prompt and in a one-token step."""
+    from trapetum_b200.csrc import ops
+    g = torch.Generator().manual_seed(5)
+    H, D, V, n = 4, 64, 64, 40
+    q = torch.randn(n, H, D, generator=g, dtype=F)
+    k = torch.randn(n, H, D, generator=g, dtype=F)
+    k = k - q * ((q * k).sum(-1, keepdim=True) / (q * q).sum(-1, keepdim=True))       # orthogonal, then a little of q
+    k = k + q * torch.where(torch.rand(n, H, 1, generator=g) < 0.5, -1e-4, 1e-4).double()
+    v, z = torch.randn(n, H, V, generator=g, dtype=F), torch.full((n, H * V), 3.0, dtype=F)
+    x = torch.cat([q.reshape(n, -1), k.reshape(n, -1), v.reshape(n, -1), z], dim=1).float()
+    want = torch.sign((x[:, :H * D].double().view(n, H, D) * x[:, H * D:2 * H * D].double().view(n, H, D)).sum(-1))
+    dec = torch.full((H,), decay, device=DEV)
+    lens = [n] if decay == 0.0 else [1] * n
+    pos = torch.zeros(n, dtype=torch.int32, device=DEV)
+    for longest in (max(lens), 0):
+        steps = [slice(0, n)] if longest or decay else [slice(i, i + 1) for i in range(n)]
+        state = torch.zeros(len(lens), H * D * V, device=DEV)
+        for sl in steps:
+            L = lens if len(steps) == 1 else [1]
+            got = ops.retention(dev(x[sl])[None].contiguous(), H, D, V, DTYPES[dtype], 0, None, 1.0, dec, 1e-12, state, pos[sl], i32(starts_of(L)),
+                                i32(seq_of(L)), i32(list(range(len(L)))), len(L), longest)
+            sign = torch.sign((got.double().cpu().view(-1, H, V) * v[sl]).sum(-1))
+            assert torch.equal(sign, want[sl])
+
+
 # ---------------------------------------------------------------------------
 # the model through the engine
 # ---------------------------------------------------------------------------

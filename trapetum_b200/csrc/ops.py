@@ -1497,7 +1497,7 @@ class _RetentionArgs(ctypes.Structure):
                 ("positions", c_void_p), ("token_seq", c_void_p), ("seq_start", c_void_p), ("slot_ids", c_void_p),
                 ("state", c_void_p), ("state_stride", c_longlong), ("rows", c_void_p), ("out", c_void_p),
                 ("batch", c_int), ("n_tokens", c_int), ("chunk_sum", c_void_p), ("chunk_hi", c_void_p), ("chunk_lo", c_void_p),
-                ("chunk_len", c_int), ("n_chunks", c_int), ("row_blocks", c_int), ("DP", c_int), ("VP", c_int)]
+                ("chunk_len", c_int), ("n_chunks", c_int), ("row_blocks", c_int), ("DP", c_int), ("VP", c_int), ("qk", c_void_p)]
 
 
 def retention_files(dtype: torch.dtype, key_dim: int, value_dim: int) -> Tuple[str, ...]:
@@ -1551,6 +1551,8 @@ def retention(part: torch.Tensor, heads: int, key_dim: int, value_dim: int, out_
             rows = torch.empty((T, heads * (2 * DP + VP)), dtype=torch.bfloat16, device=part.device)
             sums = torch.empty((batch, n_chunks, heads * DP * VP), dtype=torch.float32, device=part.device)
             halves = torch.empty((2, batch, n_chunks, heads * DP * VP), dtype=torch.bfloat16, device=part.device)
+            own = torch.empty((T, heads), dtype=torch.float32, device=part.device)
+            a.qk = own.data_ptr()
             a.rows = rows.data_ptr(); a.chunk_sum = sums.data_ptr(); a.chunk_hi = halves[0].data_ptr(); a.chunk_lo = halves[1].data_ptr()
             a.chunk_len = C; a.n_chunks = n_chunks; a.row_blocks = blocks; a.DP = DP; a.VP = VP
             _check(lib, lib.tb_retention_chunks(ctypes.byref(a), _stream()), "retention_chunks", 4)

@@ -21,8 +21,10 @@
 //
 // 32-bit: angles, rotation, decays, the state, o, its norm and the gate.  v is a product's output and is rounded to the
 // activations' dtype, as every other mixer's values are.  In the chunk form the turned q and k are rounded once, as an
-// attention kernel's are, and so are the weights (q_i . k_j) decay^(i - j) that meet v; the state and the decayed
-// keys that enter it are not: they are multiplied as sums of two bfloat16 numbers (16 bits of mantissa).
+// attention kernel's are, and so are the weights (q_i . k_j) decay^(i - j) that meet v; but a token's own product q_i . k_i
+// is taken in 32-bit from the unrounded numbers: where it is all there is (a sequence's first token) or nearly all (a
+// fast decay), the norm leaves little of it but its sign, which rounding must not turn.  The state and the decayed keys
+// that enter it are not rounded to 16 bits: they are multiplied as sums of two bfloat16 numbers (16 bits of mantissa).
 #include <cooperative_groups.h>
 #include "common.cuh"
 
@@ -43,6 +45,7 @@ struct RetentionArgs {
     int batch, n_tokens;
     float* chunk_sum; bf16* chunk_hi; bf16* chunk_lo; // chunks: [batch][n_chunks][H][DP][VP] each
     int chunk_len, n_chunks, row_blocks, DP, VP;      // DP, VP: D and V padded (64, 128, 256; multiples of 64)
+    float* qk;                                        // chunks: [T][H] every token's own q . k, in 32-bit
 };
 
 // The argument block's size, for the Python mirror's check.
@@ -281,26 +284,39 @@ __global__ void __launch_bounds__(256) retention_rows_kernel(RetentionArgs a) {
             }
             return s;
         };
-        const int dq = DP >> 2, vq = VP >> 2;
-#pragma unroll 2
-        for (int u = threadIdx.x; u < 2 * H * dq; u += blockDim.x) {
-            const int hs = u / dq, i = (u - hs * dq) << 2;
-            if (i >= half && i < 2 * half) continue;                     // made together with its partner
-            const int c = hs * D + i;                                    // the k heads follow the q heads
-            const float scale = hs < H ? 1.f : a.k_scale;
-            uint2 y = make_uint2(0u, 0u);
-            if (i < half) {
-                const float4 x = at(c), w = at(c + half), cc = *(const float4*)(cs + i), s = *(const float4*)(sn + i);
-                y = make_uint2(pack_bf16((x.x * cc.x - w.x * s.x) * scale, (x.y * cc.y - w.y * s.y) * scale),
-                               pack_bf16((x.z * cc.z - w.z * s.z) * scale, (x.w * cc.w - w.w * s.w) * scale));
-                *(uint2*)(dst + (size_t)hs * DP + i + half) =
-                    make_uint2(pack_bf16((w.x * cc.x + x.x * s.x) * scale, (w.y * cc.y + x.y * s.y) * scale),
-                               pack_bf16((w.z * cc.z + x.z * s.z) * scale, (w.w * cc.w + x.w * s.w) * scale));
-            } else if (i < D) {
-                const float4 x = at(c);
-                y = make_uint2(pack_bf16(x.x * scale, x.y * scale), pack_bf16(x.z * scale, x.w * scale));
+        const int vq = VP >> 2, lane = threadIdx.x & 31;
+        // a warp makes a head's q and k together: four numbers (and their rotation partners) of both per lane
+        for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {
+            float dot = 0.f;
+            for (int i = lane << 2; i < DP; i += 128) {
+                if (i >= half && i < 2 * half) continue;                 // made together with its partner
+                bf16* qd = dst + (size_t)h * DP + i;
+                bf16* kd = dst + (size_t)(H + h) * DP + i;
+                float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q;
+                if (i < D) { q = at(h * D + i); k = at(HD + h * D + i); }
+                if (i < half) {
+                    const float4 q2 = at(h * D + i + half), k2 = at(HD + h * D + i + half);
+                    const float4 c = *(const float4*)(cs + i), s = *(const float4*)(sn + i);
+                    auto turn = [&](float4& x, const float4& w) {
+                        const float4 lo = make_float4(x.x * c.x - w.x * s.x, x.y * c.y - w.y * s.y, x.z * c.z - w.z * s.z, x.w * c.w - w.w * s.w);
+                        const float4 hi = make_float4(w.x * c.x + x.x * s.x, w.y * c.y + x.y * s.y, w.z * c.z + x.z * s.z, w.w * c.w + x.w * s.w);
+                        x = lo;
+                        return hi;
+                    };
+                    const float4 qh = turn(q, q2);
+                    float4 kh = turn(k, k2);
+                    kh.x *= a.k_scale; kh.y *= a.k_scale; kh.z *= a.k_scale; kh.w *= a.k_scale;
+                    dot += qh.x * kh.x + qh.y * kh.y + qh.z * kh.z + qh.w * kh.w;
+                    *(uint2*)(qd + half) = make_uint2(pack_bf16(qh.x, qh.y), pack_bf16(qh.z, qh.w));
+                    *(uint2*)(kd + half) = make_uint2(pack_bf16(kh.x, kh.y), pack_bf16(kh.z, kh.w));
+                }
+                k.x *= a.k_scale; k.y *= a.k_scale; k.z *= a.k_scale; k.w *= a.k_scale;
+                dot += q.x * k.x + q.y * k.y + q.z * k.z + q.w * k.w;
+                *(uint2*)qd = make_uint2(pack_bf16(q.x, q.y), pack_bf16(q.z, q.w));
+                *(uint2*)kd = make_uint2(pack_bf16(k.x, k.y), pack_bf16(k.z, k.w));
             }
-            *(uint2*)(dst + (size_t)hs * DP + i) = y;
+            dot = warp_sum(dot);
+            if (lane == 0) a.qk[(size_t)t * H + h] = dot;
         }
 #pragma unroll 2
         for (int u = threadIdx.x; u < H * vq; u += blockDim.x) {
@@ -315,13 +331,23 @@ __global__ void __launch_bounds__(256) retention_rows_kernel(RetentionArgs a) {
             for (int sp = 1; sp < a.n_splits; sp++) s += src[(size_t)sp * a.split_stride + c];
             return s;
         };
-        for (int u = threadIdx.x; u < 2 * H * DP; u += blockDim.x) {
-            const int hs = u / DP, i = u - hs * DP, c = hs * D + i;
-            float y = 0.f;
-            if (i < half) y = at(c) * cs[i] - at(c + half) * sn[i];
-            else if (i < 2 * half) y = at(c) * cs[i - half] + at(c - half) * sn[i - half];
-            else if (i < D) y = at(c);
-            dst[u] = __float2bfloat16_rn(hs < H ? y : y * a.k_scale);
+        const int lane = threadIdx.x & 31;
+        for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {
+            float dot = 0.f;
+            for (int i = lane; i < DP; i += 32) {
+                float y[2];
+#pragma unroll
+                for (int w = 0; w < 2; w++) {
+                    const int c = (w * H + h) * D + i;
+                    y[w] = i < half ? at(c) * cs[i] - at(c + half) * sn[i]
+                         : i < 2 * half ? at(c) * cs[i - half] + at(c - half) * sn[i - half] : i < D ? at(c) : 0.f;
+                    if (w) y[w] *= a.k_scale;
+                    dst[(size_t)(w * H + h) * DP + i] = __float2bfloat16_rn(y[w]);
+                }
+                dot = fmaf(y[0], y[1], dot);
+            }
+            dot = warp_sum(dot);
+            if (lane == 0) a.qk[(size_t)t * H + h] = dot;
         }
         for (int u = threadIdx.x; u < H * VP; u += blockDim.x) {
             const int hs = u / VP, i = u - hs * VP;
@@ -543,6 +569,8 @@ __global__ void __launch_bounds__(CT) retention_out_kernel(RetentionArgs a) {
     }
     __syncthreads();                                  // the state's place takes the second tile
     const int last_row = r0 - c0 + warp * 16 + 15;    // of this warp
+    const float own_a = a.qk[(size_t)min(s0 + c0 + row_a, s0 + len - 1) * a.heads + h];
+    const float own_b = a.qk[(size_t)min(s0 + c0 + row_b, s0 + len - 1) * a.heads + h];
     for (int i = 0; i < nb; i++) {
         if (i + 1 < nb) {
             load_rows<KB, DP>(stage_of(i + 1), kb, stride, c0 + (i + 1) * KB, len);
@@ -581,7 +609,7 @@ __global__ void __launch_bounds__(CT) retention_out_kernel(RetentionArgs a) {
 #pragma unroll
                     for (int e = 0; e < 4; e++) {
                         const int dist = ((e < 2) ? row_a : row_b) - (j + (e & 1));
-                        x[e] = dist >= 0 ? s[n][e] * pw[max(dist, 0)] : 0.f;
+                        x[e] = dist > 0 ? s[n][e] * pw[max(dist, 0)] : dist == 0 ? (e < 2 ? own_a : own_b) : 0.f;
                     }
                     p[n >> 1][(n & 1) * 2] = pack_bf16(x[0], x[1]);
                     p[n >> 1][(n & 1) * 2 + 1] = pack_bf16(x[2], x[3]);
@@ -747,7 +775,7 @@ extern "C" int tb_retention_chunks(const RetentionArgs* args, cudaStream_t strea
         return tb_refuse("retention: %d chunks of %d tokens for %d row blocks", a.n_chunks, a.chunk_len, a.row_blocks);
     if ((long long)a.batch * a.n_chunks > 65535 || (long long)a.batch * a.row_blocks > 65535)
         return tb_refuse("retention: %d sequences of %d chunks exceed one launch", a.batch, a.n_chunks);
-    if (a.rows == nullptr || a.chunk_sum == nullptr || a.chunk_hi == nullptr || a.chunk_lo == nullptr)
+    if (a.rows == nullptr || a.chunk_sum == nullptr || a.chunk_hi == nullptr || a.chunk_lo == nullptr || a.qk == nullptr)
         return tb_refuse("retention: the chunk form needs its scratch");
     const int half = a.rotary_dim / 2;
     const bool vec = a.D % 4 == 0 && a.V % 4 == 0 && half % 4 == 0 && (uintptr_t)a.part % 16 == 0 && a.row_stride % 4 == 0 && a.split_stride % 4 == 0;
