@@ -54,12 +54,13 @@ struct GemmParams {
     float scale;                     // the output times this (1 for a plain product); after the cap, never with it
     int act;                         // gated epilogue: 0 gelu_tanh, 1 silu, 2 clamped_swish (only with GATED kernels)
     float limit;                     // clamped_swish: both branches are bounded by it
-    int unary;                       // plain epilogues: 0 nothing, 1 every output becomes relu(v)^2 (never on partial sums)
+    int unary;                       // plain epilogues: 0 nothing, 1 every output becomes relu(v)^2, 2 v Phi(v) (never on partial sums)
     // Grouped products (token-major tiles only): tile tp of the tokens multiplies the weight rows of group
     // tile_group[tp], which start at row tile_group[tp] * group_rows of the weight operand; a negative entry: the tile
     // is not in use and nobody touches it.  Null: one group.
     const int* tile_group;
     int group_rows;
+    const float* row_scale;          // grouped products: the sums of token row r times row_scale[r], before the activation; or null
 };
 
 // Gated epilogue.  The weight rows are interleaved in blocks of 16: [gate 0..15 | up 0..15 | gate 16..31 | ...],
@@ -106,11 +107,26 @@ template <int BN, bool SWAP, bool WIDE = false> struct Cfg {
     static constexpr int SMEM = STAGES * STAGE_BYTES + 1024 /* alignment */ + 256 /* barriers */;
 };
 
+// The exact gelu, v Phi(v), for an output that is rounded to bfloat16.  The tail Q(t) = 1 - Phi(t), t = |v|, is half of
+// erfc(t / sqrt 2), which formula 7.1.26 of Abramowitz and Stegun, Handbook of Mathematical Functions, gives as a
+// polynomial in 1 / (1 + p t / sqrt 2) times e^(-t^2 / 2) (error at most 1.5e-7).
+__device__ __forceinline__ float gelu_exact(float v) {
+    const float x = fabsf(v) * 0.70710678f;
+    const float k = __fdividef(1.0f, fmaf(0.3275911f, x, 1.0f));
+    float q = fmaf(1.061405429f, k, -1.453152027f);
+    q = fmaf(q, k, 1.421413741f);
+    q = fmaf(q, k, -0.284496736f);
+    q = fmaf(q, k, 0.254829592f);
+    q = 0.5f * q * k * __expf(-x * x);
+    return v * (v < 0.f ? q : 1.0f - q);
+}
+
 // Epilogue of token-major tiles: the thread holds CH consecutive columns (weight rows q0 .. q0 + CH - 1) of token prow.
 // What a plain epilogue does to one output before the scale: the cap, then the unary activation.
 __device__ __forceinline__ float pointwise(float v, const GemmParams& p) {
     if (p.cap > 0.f) v = softcap_f(v, p.cap);
     if (p.unary == 1) { v = fmaxf(v, 0.f); v *= v; }
+    else if (p.unary == 2) v = gelu_exact(v);
     return v;
 }
 
@@ -335,6 +351,11 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
                 tmem_ld_wait();
                 const int q0 = tq * BN + c0;                           // first row of Q in this chunk
                 if constexpr (!SWAP) {
+                    if (p.row_scale != nullptr) {
+                        const float f = prow < p.rows_p ? p.row_scale[prow] : 0.f;
+#pragma unroll
+                        for (int j = 0; j < CH; j++) r[j] = __float_as_uint(__uint_as_float(r[j]) * f);
+                    }
                     store_token_major<TOut, GATED, CH>(r, prow, q0, sp, p);
                 } else if (GATED && SWAP) {
                     // Lanes 0..15 hold gates, lanes 16..31 the ups of the same 16 features.  Two tokens a round: the
@@ -707,7 +728,7 @@ static int gemm_tc_run(const void* A, const void* W, void* C, int c_dtype, int M
                        long long lda, long long ldw, long long ldc, float softcap, int splits, float* scratch,
                        int reduce, int gated_act, float act_limit, float out_scale, int unary, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (unary < 0 || unary > 1) return tb_refuse("gemm_tc: unknown unary activation %d", unary);
+    if (unary < 0 || unary > 2) return tb_refuse("gemm_tc: unknown unary activation %d", unary);
     if (unary && (gated_act >= 0 || softcap > 0.f)) return tb_refuse("gemm_tc: a unary activation goes with neither a gate nor a cap");
     if (unary) splits = 1;                           // the activation is not linear: no partial sums
     if (!tb_gemm_tc_takes(A, W, M, N, K, lda, ldw))
@@ -743,7 +764,7 @@ static int gemm_tc_run(const void* A, const void* W, void* C, int c_dtype, int M
     else bn = N >= 256 ? 256 : 128;
 
     GemmParams p;
-    p.tile_group = nullptr; p.group_rows = 0;
+    p.tile_group = nullptr; p.group_rows = 0; p.row_scale = nullptr;
     p.K = K; p.kblocks = kblocks; p.splits = splits; p.kb_per_split = per;
     p.out = C; p.ld_out = ldc; p.partial = scratch; p.cap = splits > 1 ? 0.f : softcap;
     p.act = gated ? gated_act : 0;
@@ -810,9 +831,9 @@ static int gemm_tc_run(const void* A, const void* W, void* C, int c_dtype, int M
 // [ceil(M / 128)] group numbers in [0, groups), or -1 for a tile that is not in use (its rows of C are not written).
 static int gemm_tc_grouped_run(const void* A, const void* W, void* C, int c_dtype, int M, int N, int groups, int K,
                                long long lda, long long ldw, long long ldc, const int* tile_group, int gated_act,
-                               int unary, cudaStream_t stream) {
+                               int unary, const float* row_scale, cudaStream_t stream) {
     if (M <= 0 || N <= 0 || groups <= 0) return 0;
-    if (unary < 0 || unary > 1 || (unary && gated_act >= 0)) return tb_refuse("gemm_tc_grouped: unary activation %d (with gate %d)", unary, gated_act);
+    if (unary < 0 || unary > 2 || (unary && gated_act >= 0)) return tb_refuse("gemm_tc_grouped: unary activation %d (with gate %d)", unary, gated_act);
     if (!tb_gemm_tc_takes(A, W, M, N, K, lda, ldw))
         return tb_refuse("gemm_tc_grouped: needs K, lda, ldw multiples of 8 and 16-byte aligned operands");
     if (c_dtype != TB_F32 && c_dtype != TB_BF16) return tb_refuse("gemm_tc_grouped: unknown output dtype %d", c_dtype);
@@ -828,7 +849,7 @@ static int gemm_tc_grouped_run(const void* A, const void* W, void* C, int c_dtyp
     }
     const int bn = N >= 256 ? 256 : 128;
     GemmParams p;
-    p.tile_group = tile_group; p.group_rows = N;
+    p.tile_group = tile_group; p.group_rows = N; p.row_scale = row_scale;
     p.K = K; p.kblocks = (K + BK - 1) / BK; p.splits = 1; p.kb_per_split = p.kblocks;
     p.out = C; p.ld_out = ldc; p.partial = nullptr; p.cap = 0.f; p.scale = 1.0f;
     p.act = gated ? gated_act : 0; p.limit = 0.f; p.unary = unary;
@@ -845,14 +866,15 @@ static int gemm_tc_grouped_run(const void* A, const void* W, void* C, int c_dtyp
 extern "C" int tb_gemm_tc_grouped(const void* A, const void* W, void* C, int c_dtype, int M, int N, int groups, int K,
                                   long long lda, long long ldw, long long ldc, const int* tile_group, int gated_act,
                                   cudaStream_t stream) {
-    return gemm_tc_grouped_run(A, W, C, c_dtype, M, N, groups, K, lda, ldw, ldc, tile_group, gated_act, 0, stream);
+    return gemm_tc_grouped_run(A, W, C, c_dtype, M, N, groups, K, lda, ldw, ldc, tile_group, gated_act, 0, nullptr, stream);
 }
 
-// The grouped product whose every output becomes relu(v)^2 (unary = 1): experts without a gate branch.
-extern "C" int tb_gemm_tc_grouped_unary(const void* A, const void* W, void* C, int c_dtype, int M, int N, int groups, int K,
-                                        long long lda, long long ldw, long long ldc, const int* tile_group, int unary,
-                                        cudaStream_t stream) {
-    return gemm_tc_grouped_run(A, W, C, c_dtype, M, N, groups, K, lda, ldw, ldc, tile_group, -1, unary, stream);
+// The same with a unary activation (experts without a gate branch; 0: none) and with a number per row of A that multiplies
+// its sums before any activation (row_scale [M], or null).
+extern "C" int tb_gemm_tc_grouped_ex(const void* A, const void* W, void* C, int c_dtype, int M, int N, int groups, int K,
+                                     long long lda, long long ldw, long long ldc, const int* tile_group, int gated_act, int unary,
+                                     const float* row_scale, cudaStream_t stream) {
+    return gemm_tc_grouped_run(A, W, C, c_dtype, M, N, groups, K, lda, ldw, ldc, tile_group, gated_act, unary, row_scale, stream);
 }
 
 extern "C" int tb_gemm_tc_ex(const void* A, const void* W, void* C, int c_dtype, int M, int N, int K,
@@ -861,7 +883,7 @@ extern "C" int tb_gemm_tc_ex(const void* A, const void* W, void* C, int c_dtype,
     return gemm_tc_run(A, W, C, c_dtype, M, N, K, lda, ldw, ldc, softcap, splits, scratch, reduce, gated_act, act_limit, out_scale, 0, stream);
 }
 
-// The plain product whose every output becomes relu(v)^2 (unary = 1): a feed-forward without a gate branch.
+// The plain product whose every output becomes relu(v)^2 (unary = 1) or v Phi(v) (2): a feed-forward without a gate branch.
 extern "C" int tb_gemm_tc_unary(const void* A, const void* W, void* C, int c_dtype, int M, int N, int K,
                                 long long lda, long long ldw, long long ldc, int unary, cudaStream_t stream) {
     return gemm_tc_run(A, W, C, c_dtype, M, N, K, lda, ldw, ldc, 0.f, 1, nullptr, 0, -1, 0.f, 1.0f, unary, stream);

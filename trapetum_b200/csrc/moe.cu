@@ -5,12 +5,15 @@
 //                    experts form `groups` equal groups of neighbours, a group's score is the sum of its
 //                    `group_top` largest choice scores, experts outside the `keep` best groups cannot be chosen
 //                    (their choice scores count as minus infinity); the `top` largest choice scores win (the
-//                    lower index on a tie); weights are the winners' s divided by their sum + eps, times out_scale.  Also the
+//                    lower index on a tie); weights are the winners' s divided by their sum + eps (or undivided), times out_scale.  Also the
 //                    shared expert's gate sigmoid(g . x), one number per token, if asked for.
 //   tb_moe_gate_up   for every (token, chosen expert): silu(G_e x) * (U_e x), or, for experts without a gate matrix,
 //                    relu(U_e x)^2
 //   tb_moe_down      out[t] = sum_k weight[t,k] * D_e(t,k) a[t,k]  (+ gate[t] * shared[t], the shared expert's output
 //                    given as 32-bit split-K partial sums), 32-bit
+//
+// The weight may multiply what the expert reads instead of what it returns (weight_in): silu(w G_e x) * (w U_e x) and no
+// weight in the sum.  The products are linear, so it is their 32-bit sums (or the 32-bit copy of x) that are multiplied.
 //
 // The router is 32-bit throughout.  The experts' products take operands of the activations' dtype and sum in
 // 32-bit; a[t,k] is rounded to the activations' dtype, the weighted sum over the experts is not.
@@ -29,7 +32,9 @@ struct MoeRouteArgs {
     int softmax;                               // scores are softmax(z) over the experts instead of sigmoid(z)
     float out_scale;                           // the weights times this
     const float* bias;                         // [E] added to the logits themselves, or null
+    int raw_scores;                            // the weights are the winners' scores themselves: no division by their sum
 };
+extern "C" int tb_moe_route_args_bytes() { return (int)sizeof(MoeRouteArgs); }      // for the Python mirror's check
 
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 #pragma unroll
@@ -127,7 +132,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
         }
     }
     __syncwarp();
-    const float inv = a.out_scale / (wsum + a.weight_eps);
+    const float inv = a.raw_scores ? a.out_scale : a.out_scale / (wsum + a.weight_eps);
     for (int n = lane; n < a.top; n += 32) a.weight[(size_t)t * a.top + n] *= inv;
 }
 
@@ -142,7 +147,9 @@ struct MoeExpertArgs {
     float* out;                                // [T][W]
     int n_tokens, W, ff, top;
     int ungated;                               // experts are D relu(U x)^2: there is no gate matrix
+    int weight_in;                             // the weight multiplies x, not the expert's output
 };
+extern "C" int tb_moe_expert_args_bytes() { return (int)sizeof(MoeExpertArgs); }    // for the Python mirror's check
 
 // n numbers of the activations' dtype into shared memory as 32-bit, times `scale`, by all threads of the block: 16 bytes
 // a load where the dtype is 16-bit, n a multiple of 8 and the source 16-byte aligned.
@@ -226,7 +233,7 @@ __global__ void __launch_bounds__(256) moe_gate_up_kernel(MoeExpertArgs a) {
     pdl_wait();
     const int e = a.idx[pair];
     const T* x = (const T*)a.x + (size_t)t * a.x_stride;
-    fill_f32<T>(x_s, x, a.W, 1.f);
+    fill_f32<T>(x_s, x, a.W, a.weight_in ? a.weight[pair] : 1.f);
     __syncthreads();
     const T* gw = (const T*)a.gate_w + (size_t)e * a.ff * a.W;
     const T* uw = (const T*)a.up_w + (size_t)e * a.ff * a.W;
@@ -253,7 +260,8 @@ __global__ void __launch_bounds__(256) moe_down_kernel(MoeExpertArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarp = blockDim.x >> 5;
     pdl_wait();
     for (int k = 0; k < a.top; k++)
-        fill_f32<T>(a_s + (size_t)k * a.ff, (const T*)a.act + ((size_t)t * a.top + k) * a.ff, a.ff, a.weight[(size_t)t * a.top + k]);
+        fill_f32<T>(a_s + (size_t)k * a.ff, (const T*)a.act + ((size_t)t * a.top + k) * a.ff, a.ff,
+                    a.weight_in ? 1.f : a.weight[(size_t)t * a.top + k]);
     __syncthreads();
     for (int c0 = (blockIdx.y * nwarp + warp) * MV_ROWS; c0 < a.W; c0 += gridDim.y * nwarp * MV_ROWS) {
         const int nr = min(MV_ROWS, a.W - c0);
@@ -356,7 +364,9 @@ struct MoeGroupedArgs {
     bf16* act;                                        // [P][ff]
     float* pair_out;                                  // [P][W]
     int W, ff, top;
+    int weight_in;                                    // the weight multiplies the first product's sums, not the second's
 };
+extern "C" int tb_moe_grouped_args_bytes() { return (int)sizeof(MoeGroupedArgs); }  // for the Python mirror's check
 
 // MODE 1: rows of x (by pair / top) times [G_e ; U_e] for 64 columns of ff, then silu(g) * u  ->  act[pair]
 // MODE 2: rows of x (by pair / top) times U_e for 128 columns of ff, then relu(u)^2            ->  act[pair]
@@ -440,6 +450,11 @@ __global__ void __launch_bounds__(MG_THREADS, 2) moe_grouped_kernel(MoeGroupedAr
     for (int m = 0; m < 2; m++) {
         const int ra = wm * 32 + m * 16 + (lane >> 2), rb = ra + 8;
         const int pa = row_src[ra], pb = row_src[rb];
+        if (FROM_X && a.weight_in) {
+            const float ia = pa >= 0 ? a.weight[pa] : 0.f, ib = pb >= 0 ? a.weight[pb] : 0.f;
+#pragma unroll
+            for (int n = 0; n < 8; n++) { acc[m][n][0] *= ia; acc[m][n][1] *= ia; acc[m][n][2] *= ib; acc[m][n][3] *= ib; }
+        }
         if (GATED) {
 #pragma unroll
             for (int n = 0; n < 4; n++) {
@@ -465,7 +480,7 @@ __global__ void __launch_bounds__(MG_THREADS, 2) moe_grouped_kernel(MoeGroupedAr
                 }
             }
         } else {
-            const float wa = pa >= 0 ? a.weight[pa] : 0.f, wb = pb >= 0 ? a.weight[pb] : 0.f;
+            const float wa = a.weight_in ? 1.f : pa >= 0 ? a.weight[pa] : 0.f, wb = a.weight_in ? 1.f : pb >= 0 ? a.weight[pb] : 0.f;
 #pragma unroll
             for (int n = 0; n < 8; n++) {
 #pragma unroll
@@ -502,7 +517,8 @@ __global__ void moe_sum_pairs_kernel(const float* __restrict__ pair_out, const f
 // The same grouping for the tcgen05 product (gemm_tc.cu, grouped mode): the pairs are laid out expert by expert
 // with every expert's stretch padded to whole tiles of 128 rows, so that a tile of the product's token operand
 // belongs to one expert.  tb_moe_group_padded makes the layout (where every pair goes, which pair every row
-// holds, every tile's expert), tb_moe_gather_rows fills the operand, and tb_moe_combine_sorted adds a token's
+// holds, every tile's expert), tb_moe_gather_rows fills the operand (and, if asked for, lays every row's weight out
+// beside it, for weights that multiply the experts' input), and tb_moe_combine_sorted adds a token's
 // weighted expert outputs (and the shared expert) back up.
 // ---------------------------------------------------------------------------
 struct MoePadArgs {
@@ -539,11 +555,13 @@ __global__ void __launch_bounds__(1024) moe_group_padded_kernel(MoePadArgs a) {
 }
 
 __global__ void __launch_bounds__(128) moe_gather_rows_kernel(const bf16* __restrict__ x, long long x_stride, const int* __restrict__ row_pair,
-                                                              bf16* __restrict__ out, int W, int top) {
+                                                              bf16* __restrict__ out, int W, int top,
+                                                              const float* __restrict__ weight, float* __restrict__ row_weight) {
     pdl_launch_dependents();
     pdl_wait();
     const int r = blockIdx.x;
     const int p = row_pair[r];
+    if (row_weight != nullptr && threadIdx.x == 0) row_weight[r] = p < 0 ? 0.f : weight[p];
     uint4* dst = (uint4*)(out + (size_t)r * W);
     if (p < 0) { for (int c = threadIdx.x; c < W / 8; c += blockDim.x) dst[c] = make_uint4(0, 0, 0, 0); return; }
     const uint4* src = (const uint4*)(x + (size_t)(p / top) * x_stride);
@@ -559,7 +577,7 @@ __global__ void moe_combine_sorted_kernel(const float* __restrict__ y, const int
     if (i >= n) return;
     const long long t = i / W; const int c = (int)(i % W);
     float acc = 0.f;
-    for (int k = 0; k < top; k++) acc = fmaf(weight[t * top + k], y[(size_t)pos[t * top + k] * W + c], acc);   // in the order of the choice
+    for (int k = 0; k < top; k++) acc = fmaf(weight != nullptr ? weight[t * top + k] : 1.f, y[(size_t)pos[t * top + k] * W + c], acc);   // in the order of the choice
     if (shared != nullptr) {
         float sh = 0.f;
         for (int s = 0; s < shared_splits; s++) sh += shared[(size_t)s * shared_split_stride + i];
@@ -577,10 +595,12 @@ extern "C" int tb_moe_group_padded(const MoePadArgs* args, cudaStream_t stream) 
 }
 
 extern "C" int tb_moe_gather_rows(const void* x, long long x_stride, const int* row_pair, void* out, int rows, int W, int top,
-                                  cudaStream_t stream) {
+                                  const float* weight, float* row_weight, cudaStream_t stream) {
     if (rows <= 0) return 0;
+    if (row_weight != nullptr && weight == nullptr) return tb_refuse("moe_gather_rows: no weights to lay out");
     if (W % 8 || x_stride % 8 || ((uintptr_t)x & 15) || ((uintptr_t)out & 15)) return tb_refuse("moe_gather_rows: rows must be 16-byte aligned");
-    tb_launch(moe_gather_rows_kernel, dim3(rows), dim3(128), 0, stream, (const bf16*)x, x_stride, row_pair, (bf16*)out, W, top);
+    tb_launch(moe_gather_rows_kernel, dim3(rows), dim3(128), 0, stream, (const bf16*)x, x_stride, row_pair, (bf16*)out, W, top,
+              weight, row_weight);
     return tb_launch_status();
 }
 

@@ -82,7 +82,9 @@ def args_mirrors():
     """(library, function that returns the C side's size, Python structure) of the argument blocks that have such a
     function: a mirror that has drifted from its C struct makes a kernel read garbage pointers."""
     return (("gla", "tb_gla_args_bytes", _GlaArgs), ("retention", "tb_retention_args_bytes", _RetentionArgs),
-            ("projnorm_kv", "tb_projnorm_kv_args_bytes", _ProjNormKvArgs), ("norm", "tb_add_terms_args_bytes", _AddTermsArgs))
+            ("projnorm_kv", "tb_projnorm_kv_args_bytes", _ProjNormKvArgs), ("norm", "tb_add_terms_args_bytes", _AddTermsArgs),
+            ("dyt", "tb_dyt_args_bytes", _DytArgs), ("moe", "tb_moe_route_args_bytes", _MoeRouteArgs),
+            ("moe", "tb_moe_expert_args_bytes", _MoeExpertArgs), ("moe", "tb_moe_grouped_args_bytes", _MoeGroupedArgs))
 
 
 def _rows_contig(t: torch.Tensor, what: str) -> None:
@@ -303,9 +305,67 @@ def cast(x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
     return out
 
 
+class _DytArgs(ctypes.Structure):
+    _fields_ = [("h", c_void_p), ("a", c_void_p), ("n_splits", c_int), ("split_stride", c_longlong),
+                ("alpha_a", c_float), ("wa", c_void_p), ("ba", c_void_p), ("alpha_b", c_float), ("wb", c_void_p), ("bb", c_void_p),
+                ("out", c_void_p), ("out_stride", c_longlong), ("take", c_int), ("give", c_int), ("from_a", c_int),
+                ("rows", c_int), ("width", c_int)]
+
+
+def dyt(h: Optional[torch.Tensor], a: Optional[torch.Tensor] = None, norm_a=None, norm_b=None,
+        out_dtype: Optional[torch.dtype] = None, replace: bool = False, out: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """Dynamic tanh norms around the residual sum (see dyt.cu).  A norm is ``(alpha, w, b)``: a number and two float32
+    vectors of the row width, ``tanh(alpha x) w + b``.
+
+    ``h`` (float32, in place): with ``a`` and ``norm_a``, ``h += norm_a(a)``; with ``a`` and ``replace``, ``h <- a``; without
+    ``a`` it stays.  ``a`` is [rows, width], or float32 partial sums [splits, rows, width].  ``h`` None: ``norm_b(a)`` alone.
+    With ``norm_b`` returns ``norm_b(h)`` in ``out_dtype``; with ``out`` (rows of the width, possibly a column slice of a
+    wider matrix) writes ``norm_b(h)``, or without ``norm_b`` ``h`` itself, into it."""
+    vectors = [t for n in (norm_a, norm_b) if n is not None for t in n[1:]]
+    _cuda(h, a, out, *vectors)
+    x = h if h is not None else a
+    rows, width = x.shape[-2], x.shape[-1]
+    if h is not None and (h.dtype != torch.float32 or h.dim() != 2 or not h.is_contiguous()):
+        raise KernelError("dyt: the residual stream must be contiguous float32 [rows, width]")
+    for t in vectors:
+        if t.dtype != torch.float32 or t.numel() != width or not t.is_contiguous():
+            raise KernelError(f"dyt: a norm's weight and bias must be contiguous float32 [{width}]")
+    args = _DytArgs()
+    args.rows = rows; args.width = width; args.n_splits = 1; args.from_a = int(h is None)
+    args.h = h.data_ptr() if h is not None else None
+    if a is not None:
+        if a.dim() == 3:
+            if a.dtype != torch.float32 or tuple(a.shape[1:]) != (rows, width) or a.stride(1) != width or a.stride(2) != 1:
+                raise KernelError(f"dyt: partial sums must be float32 [splits, {rows}, {width}], got {tuple(a.shape)} {a.dtype}")
+            args.n_splits = a.shape[0]; args.split_stride = a.stride(0)
+        elif tuple(a.shape) != (rows, width) or not a.is_contiguous():
+            raise KernelError(f"dyt: branch {tuple(a.shape)} does not fit rows of {width}")
+        args.a = a.data_ptr()
+    if h is not None:
+        args.take = 0 if a is None else 2 if replace else 1
+        if args.take == 1 and norm_a is None:
+            raise KernelError("dyt: a branch that is added needs its norm")
+    if norm_a is not None:
+        args.alpha_a = norm_a[0]; args.wa = norm_a[1].data_ptr(); args.ba = norm_a[2].data_ptr()
+    if norm_b is not None:
+        args.alpha_b = norm_b[0]; args.wb = norm_b[1].data_ptr(); args.bb = norm_b[2].data_ptr()
+        if out is None:
+            out = torch.empty((rows, width), dtype=out_dtype, device=x.device)
+    if out is not None:
+        if tuple(out.shape) != (rows, width) or out.stride(1) != 1:
+            raise KernelError(f"dyt: the output must be [{rows}, {width}] with contiguous rows, got {tuple(out.shape)}")
+        args.out = out.data_ptr(); args.out_stride = out.stride(0); args.give = 1 if norm_b is not None else 2
+    lib = build.load("dyt")
+    _check(lib, lib.tb_dyt(ctypes.byref(args), c_int(code(a.dtype) if a is not None else 0),
+                           c_int(code(out.dtype) if out is not None else 0), _stream()), "dyt")
+    return out
+
+
 # ---------------------------------------------------------------------------
 ACTIVATIONS = {"gelu_tanh": 0, "silu": 1, "clamped_swish": 2}
-UNARY_ACTIVATIONS = {"relu2": 3}          # activations of a feed-forward without a gate branch: relu2(u) = relu(u)^2
+# activations of a feed-forward without a gate branch: relu2(u) = relu(u)^2, gelu(u) = u Phi(u) with the normal
+# distribution's Phi itself (no tanh in its place)
+UNARY_ACTIVATIONS = {"relu2": 3, "gelu": 4}
 ACTIVATIONS_WITH_LIMIT = ("clamped_swish",)
 
 
@@ -531,7 +591,7 @@ class _ProjNormKvArgs(ctypes.Structure):
                 ("positions", c_void_p), ("token_seq", c_void_p), ("len_after", c_void_p),
                 ("k_pool", c_void_p), ("v_pool", c_void_p), ("page_table", c_void_p), ("pt_stride", c_int),
                 ("page_rows", c_int), ("ring_rows", c_int), ("bias", c_void_p), ("head_norm", c_int), ("v_first", c_void_p),
-                ("v_lam", c_float), ("v_keep", c_void_p)]
+                ("v_lam", c_float), ("v_keep", c_void_p), ("rot_mult", c_float)]
 
 
 def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, vdim: int, padded: int,
@@ -540,7 +600,8 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
                 positions: torch.Tensor, token_seq: torch.Tensor, len_after: torch.Tensor,
                 k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], page_table: Optional[torch.Tensor],
                 ring_rows: int, bias: Optional[torch.Tensor] = None, head_norm: bool = False,
-                v_first: Optional[torch.Tensor] = None, v_lam: float = 0.0, v_keep: Optional[torch.Tensor] = None):
+                v_first: Optional[torch.Tensor] = None, v_lam: float = 0.0, v_keep: Optional[torch.Tensor] = None,
+                rot_mult: float = 1.0):
     """From the q/k/v(/gate) product's float32 partial sums [splits, T, H dim + G dim + G vdim (+ H)] to
     ([T, (H + 2 G) * padded] in ``out_dtype``, sigmoid of the gate columns float32 [T, H] or None): q and k divided by
     their root mean square over the whole projection times ``q_norm_w`` / ``k_norm_w`` (float32; None: no norm), q heads
@@ -550,7 +611,7 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
     up to a multiple of four), added to the summed row before anything else.  ``n_kv_heads`` 0: the product holds
     queries only.  ``head_norm``: the norms are per head, with weights of ``dim`` numbers that the heads share.
     ``v_first`` (float32 [T, G vdim]): the values become ``(1 - v_lam) v + v_lam v_first``; ``v_keep`` (the same shape)
-    receives this product's own values in 32-bit."""
+    receives this product's own values in 32-bit.  ``rot_mult`` multiplies the rotation's cos and sin."""
     _cuda(v_first, v_keep)
     for name, t in (("v_first", v_first), ("v_keep", v_keep)):
         if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != (partial.shape[1], n_kv_heads * vdim) or not t.is_contiguous()):
@@ -597,7 +658,7 @@ def projnorm_kv(partial: torch.Tensor, n_heads: int, n_kv_heads: int, dim: int, 
     a.pt_stride = page_table.stride(0) if k_pool is not None else 0
     a.page_rows = PAGE_ROWS; a.ring_rows = ring_rows
     a.bias = bias.data_ptr() if bias is not None else None
-    a.head_norm = int(bool(head_norm)); a.v_lam = v_lam
+    a.head_norm = int(bool(head_norm)); a.v_lam = v_lam; a.rot_mult = rot_mult
     a.v_first = v_first.data_ptr() if v_first is not None else None
     a.v_keep = v_keep.data_ptr() if v_keep is not None else None
     lib = build.load("projnorm_kv")
@@ -887,6 +948,7 @@ def gemm_tc_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 GEMM_TC_GATES = ("gelu_tanh", "silu", "clamped_swish")
+GEMM_TC_UNARY = {"relu2": 1, "gelu": 2}      # unary activations the epilogue applies, by its own codes
 
 
 def gemm_tc_gates(activation: str) -> bool:
@@ -905,17 +967,17 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, softcap: f
     ``gated_act`` ("gelu_tanh" or "silu"): ``w`` holds gate and up rows interleaved in blocks of 16
     (see :func:`interleave_gate_up`); the result is bfloat16 [M, N/2] = act(gate) * up, taken on the
     32-bit accumulators in the epilogue ("clamped_swish" takes ``act_limit``).  ``out_scale``: the result times this
-    number (not with a cap, a gate or partial sums).  ``unary_act`` ("relu2"): every output becomes act(output), taken
+    number (not with a cap, a gate or partial sums).  ``unary_act`` ("relu2", "gelu"): every output becomes act(output), taken
     on the 32-bit accumulators (no partial sums, no cap, no gate)."""
     _cuda(a, w, out)
     if unary_act is not None:
-        if unary_act not in UNARY_ACTIVATIONS or partials or softcap or gated_act is not None or out_scale != 1.0 or not gemm_tc_takes(a, w):
-            raise KernelError(f"gemm_tc: the unary epilogue knows {sorted(UNARY_ACTIVATIONS)} and takes no partials, cap, gate or scale")
+        if unary_act not in GEMM_TC_UNARY or partials or softcap or gated_act is not None or out_scale != 1.0 or not gemm_tc_takes(a, w):
+            raise KernelError(f"gemm_tc: the unary epilogue knows {sorted(GEMM_TC_UNARY)} and takes no partials, cap, gate or scale")
         out = torch.empty((a.shape[0], w.shape[0]), dtype=out_dtype, device=a.device)
         lib = build.load("gemm_tc")
         _check(lib, lib.tb_gemm_tc_unary(_ptr(a), _ptr(w), _ptr(out), c_int(code(out_dtype)), c_int(a.shape[0]), c_int(w.shape[0]),
                                          c_int(a.shape[1]), c_longlong(a.stride(0)), c_longlong(w.stride(0)),
-                                         c_longlong(out.stride(0)), c_int(1), _stream()), "gemm_tc")
+                                         c_longlong(out.stride(0)), c_int(GEMM_TC_UNARY[unary_act]), _stream()), "gemm_tc")
         return out
     if not gemm_tc_takes(a, w):
         raise KernelError(f"gemm_tc does not take a {tuple(a.shape)}/{a.stride()} {a.dtype}, "
@@ -1841,16 +1903,18 @@ class _MoeRouteArgs(ctypes.Structure):
     _fields_ = [("logits", c_void_p), ("splits", c_int), ("split_stride", c_longlong), ("row_stride", c_longlong),
                 ("correction", c_void_p), ("has_gate", c_int), ("idx", c_void_p), ("weight", c_void_p), ("gate", c_void_p),
                 ("n_tokens", c_int), ("W", c_int), ("E", c_int), ("top", c_int), ("groups", c_int), ("keep", c_int),
-                ("group_top", c_int), ("weight_eps", c_float), ("softmax", c_int), ("out_scale", c_float), ("bias", c_void_p)]
+                ("group_top", c_int), ("weight_eps", c_float), ("softmax", c_int), ("out_scale", c_float), ("bias", c_void_p),
+                ("raw_scores", c_int)]
 
 
 def moe_route(logits: torch.Tensor, experts: int, correction: Optional[torch.Tensor], has_gate: bool,
               top: int, groups: int, keep: int, group_top: int, weight_eps: float, score: str = "sigmoid",
-              out_scale: float = 1.0, bias: Optional[torch.Tensor] = None):
+              out_scale: float = 1.0, bias: Optional[torch.Tensor] = None, renormalize: bool = True):
     """Routing with groups (see moe.cu; ``score`` "sigmoid" or "softmax" over all experts; the weights come times
     ``out_scale``) from the router's logits: float32 [T, >= experts (+ 1)] or
     partial sums [splits, T, ...] of the router product (column ``experts`` is the shared expert's gate product if
     ``has_gate``).  ``bias``: float32 [experts] added to the logits themselves (``correction`` only steers the choice).
+    ``renormalize`` False: the weights are the winners' scores as they are, not their shares of the winners' sum.
     Returns (chosen experts int32 [T, top], their weights float32 [T, top], the shared expert's gate
     float32 [T] or None)."""
     _cuda(logits, correction, bias)
@@ -1878,6 +1942,7 @@ def moe_route(logits: torch.Tensor, experts: int, correction: Optional[torch.Ten
         raise KernelError(f"moe_route: scores are 'sigmoid' or 'softmax', not '{score}'")
     a.softmax = int(score == "softmax"); a.out_scale = out_scale
     a.bias = bias.data_ptr() if bias is not None else None
+    a.raw_scores = int(not renormalize)
     lib = build.load("moe")
     _check(lib, lib.tb_moe_route(ctypes.byref(a), _stream()), "moe_route")
     return idx, weight, gate
@@ -1892,10 +1957,11 @@ class _MoePadArgs(ctypes.Structure):
                 ("P", c_int), ("E", c_int), ("max_rows", c_int)]
 
 
-def _moe_grouped_tc(x, gate_up_w, down_w, idx, weight, shared, gate, out, ungated=False):
+def _moe_grouped_tc(x, gate_up_w, down_w, idx, weight, shared, gate, out, ungated=False, on_input=False):
     """The experts' products on the tcgen05 kernel: the pairs ordered by expert, each expert's stretch padded to whole
     tiles of 128 rows (see moe.cu and gemm_tc.cu's grouped mode).  Shapes depend on the sizes only.  ``ungated``:
-    ``gate_up_w`` holds the up rows alone and the first product's epilogue is relu(u)^2."""
+    ``gate_up_w`` holds the up rows alone and the first product's epilogue is relu(u)^2.  ``on_input``: a pair's weight
+    multiplies the first product's sums (the gather lays it out beside the rows) instead of the second's."""
     T, W = x.shape
     E, ff2 = gate_up_w.shape[0], gate_up_w.shape[1]
     ff = ff2 if ungated else ff2 // 2
@@ -1910,23 +1976,20 @@ def _moe_grouped_tc(x, gate_up_w, down_w, idx, weight, shared, gate, out, ungate
     g.P = P; g.E = E; g.max_rows = max_rows
     _check(lib, lib.tb_moe_group_padded(ctypes.byref(g), _stream()), "moe_group_padded")
     xs = torch.empty((max_rows, W), dtype=x.dtype, device=x.device)
+    row_weight = torch.empty(max_rows, dtype=torch.float32, device=x.device) if on_input else None
     _check(lib, lib.tb_moe_gather_rows(_ptr(x), c_longlong(x.stride(0)), _ptr(row_pair), _ptr(xs), c_int(max_rows), c_int(W),
-                                       c_int(top), _stream()), "moe_gather_rows")
+                                       c_int(top), _ptr(weight if on_input else None), _ptr(row_weight), _stream()), "moe_gather_rows")
     act = torch.empty((max_rows, ff), dtype=x.dtype, device=x.device)
     y = torch.empty((max_rows, W), dtype=torch.float32, device=x.device)
     gl = build.load("gemm_tc")
-    if ungated:
-        _check(gl, gl.tb_gemm_tc_grouped_unary(_ptr(xs), _ptr(gate_up_w), _ptr(act), c_int(code(x.dtype)), c_int(max_rows), c_int(ff),
-                                               c_int(E), c_int(W), c_longlong(W), c_longlong(W), c_longlong(ff), _ptr(tile_group),
-                                               c_int(1), _stream()), "gemm_tc_grouped")
-    else:
-        _check(gl, gl.tb_gemm_tc_grouped(_ptr(xs), _ptr(gate_up_w), _ptr(act), c_int(code(x.dtype)), c_int(max_rows), c_int(ff2),
-                                         c_int(E), c_int(W), c_longlong(W), c_longlong(W), c_longlong(ff), _ptr(tile_group),
-                                         c_int(ACTIVATIONS["silu"]), _stream()), "gemm_tc_grouped")
+    _check(gl, gl.tb_gemm_tc_grouped_ex(_ptr(xs), _ptr(gate_up_w), _ptr(act), c_int(code(x.dtype)), c_int(max_rows), c_int(ff2),
+                                        c_int(E), c_int(W), c_longlong(W), c_longlong(W), c_longlong(ff), _ptr(tile_group),
+                                        c_int(-1 if ungated else ACTIVATIONS["silu"]), c_int(GEMM_TC_UNARY["relu2"] if ungated else 0),
+                                        _ptr(row_weight), _stream()), "gemm_tc_grouped")
     _check(gl, gl.tb_gemm_tc_grouped(_ptr(act), _ptr(down_w), _ptr(y), c_int(code(torch.float32)), c_int(max_rows), c_int(W),
                                      c_int(E), c_int(ff), c_longlong(ff), c_longlong(ff), c_longlong(W), _ptr(tile_group),
                                      c_int(-1), _stream()), "gemm_tc_grouped")
-    _check(lib, lib.tb_moe_combine_sorted(_ptr(y), _ptr(pos), _ptr(weight), _ptr(shared),
+    _check(lib, lib.tb_moe_combine_sorted(_ptr(y), _ptr(pos), _ptr(None if on_input else weight), _ptr(shared),
                                           c_int(shared.shape[0] if shared is not None else 0),
                                           c_longlong(shared.stride(0) if shared is not None else 0), _ptr(gate), _ptr(out),
                                           c_int(T), c_int(W), c_int(top), _stream()), "moe_combine_sorted")
@@ -1942,10 +2005,10 @@ class _MoeGroupedArgs(ctypes.Structure):
     _fields_ = [("x", c_void_p), ("x_stride", c_longlong), ("gate_w", c_void_p), ("up_w", c_void_p), ("down_w", c_void_p),
                 ("perm", c_void_p), ("tile_expert", c_void_p), ("tile_row0", c_void_p), ("tile_rows", c_void_p),
                 ("n_tiles", c_void_p), ("weight", c_void_p), ("act", c_void_p), ("pair_out", c_void_p),
-                ("W", c_int), ("ff", c_int), ("top", c_int)]
+                ("W", c_int), ("ff", c_int), ("top", c_int), ("weight_in", c_int)]
 
 
-def _moe_grouped(x, gate_w, up_w, down_w, idx, weight, shared, gate, out):
+def _moe_grouped(x, gate_w, up_w, down_w, idx, weight, shared, gate, out, on_input=False):
     """The experts' products with the pairs grouped by expert (bfloat16, tensor cores; see moe.cu).  The grid holds the
     most tiles there can be, so nothing the host does depends on which experts were chosen."""
     T, W = x.shape
@@ -1968,7 +2031,7 @@ def _moe_grouped(x, gate_w, up_w, down_w, idx, weight, shared, gate, out):
     a.gate_w = gate_w.data_ptr() if gate_w is not None else None; a.up_w = up_w.data_ptr(); a.down_w = down_w.data_ptr()
     a.perm = perm.data_ptr(); a.tile_expert = te.data_ptr(); a.tile_row0 = tr0.data_ptr(); a.tile_rows = trn.data_ptr()
     a.n_tiles = nt.data_ptr(); a.weight = weight.data_ptr(); a.act = act.data_ptr(); a.pair_out = pair_out.data_ptr()
-    a.W = W; a.ff = ff; a.top = top
+    a.W = W; a.ff = ff; a.top = top; a.weight_in = int(on_input)
     _check(lib, lib.tb_moe_grouped(ctypes.byref(a), _ptr(shared), c_int(shared.shape[0] if shared is not None else 0),
                                    c_longlong(shared.stride(0) if shared is not None else 0), _ptr(gate), _ptr(out), c_int(T),
                                    c_int(max_tiles), _stream()), "moe_grouped", 3)
@@ -1979,17 +2042,22 @@ class _MoeExpertArgs(ctypes.Structure):
     _fields_ = [("x", c_void_p), ("x_stride", c_longlong), ("gate_w", c_void_p), ("up_w", c_void_p), ("down_w", c_void_p),
                 ("idx", c_void_p), ("weight", c_void_p), ("act", c_void_p), ("shared", c_void_p), ("shared_splits", c_int),
                 ("shared_split_stride", c_longlong), ("gate", c_void_p), ("out", c_void_p),
-                ("n_tokens", c_int), ("W", c_int), ("ff", c_int), ("top", c_int), ("ungated", c_int)]
+                ("n_tokens", c_int), ("W", c_int), ("ff", c_int), ("top", c_int), ("ungated", c_int), ("weight_in", c_int)]
 
 
 def moe_experts(x: torch.Tensor, gate_w: Optional[torch.Tensor], up_w: torch.Tensor, down_w: torch.Tensor, idx: torch.Tensor,
                 weight: torch.Tensor, shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
-                gate_up_w: Optional[torch.Tensor] = None) -> torch.Tensor:
+                gate_up_w: Optional[torch.Tensor] = None, weight_on: str = "output") -> torch.Tensor:
     """The weighted sum of every token's chosen experts ``down_e(silu(gate_e x) * up_e x)`` plus ``gate[t] * shared[t]``
     (``shared`` float32 partial sums [splits, T, W]); returns float32 [T, W].  Expert matrices: ``gate_w``, ``up_w``
     [E, ff, W] and ``down_w`` [E, W, ff] of x's dtype; ``gate_up_w`` [E, 2 ff, W]: every expert's gate and up rows
     interleaved (``interleave_gate_up``), which lets many tokens run on the tcgen05 product.  ``gate_w`` None: the
-    experts have no gate matrix and are ``down_e(relu(up_e x)^2)``."""
+    experts have no gate matrix and are ``down_e(relu(up_e x)^2)``.  ``weight_on`` "input": a winner's weight w multiplies
+    what its expert reads, ``down_e(silu(w gate_e x) * w up_e x)``, and not what it returns (the first products are
+    linear, so their 32-bit sums are multiplied)."""
+    if weight_on not in ("input", "output"):
+        raise KernelError(f"moe: weights go on the experts' 'input' or 'output', not '{weight_on}'")
+    on_input = weight_on == "input"
     _cuda(x, gate_w, up_w, down_w, idx, weight, shared, gate, gate_up_w)
     _rows_contig(x, "moe: x")
     T, W = x.shape
@@ -2011,15 +2079,15 @@ def moe_experts(x: torch.Tensor, gate_w: Optional[torch.Tensor], up_w: torch.Ten
     if x.dtype == torch.bfloat16 and T * top >= MOE_GROUPED_FROM and W % 8 == 0 and ff % 8 == 0 and x.stride(0) % 8 == 0 \
             and x.data_ptr() % 16 == 0:
         if ungated and T * top >= MOE_TCGEN05_FROM:
-            return _moe_grouped_tc(x, up_w, down_w, idx, weight, shared, gate, out, ungated=True)
+            return _moe_grouped_tc(x, up_w, down_w, idx, weight, shared, gate, out, ungated=True, on_input=on_input)
         if gate_up_w is not None and T * top >= MOE_TCGEN05_FROM and ff % 16 == 0:
-            return _moe_grouped_tc(x, gate_up_w, down_w, idx, weight, shared, gate, out)
-        return _moe_grouped(x, gate_w, up_w, down_w, idx, weight, shared, gate, out)
+            return _moe_grouped_tc(x, gate_up_w, down_w, idx, weight, shared, gate, out, on_input=on_input)
+        return _moe_grouped(x, gate_w, up_w, down_w, idx, weight, shared, gate, out, on_input)
     act = torch.empty((T * top, ff), dtype=x.dtype, device=x.device)
     a = _MoeExpertArgs()
     a.x = x.data_ptr(); a.x_stride = x.stride(0)
     a.gate_w = gate_w.data_ptr() if gate_w is not None else None; a.up_w = up_w.data_ptr(); a.down_w = down_w.data_ptr()
-    a.ungated = int(ungated)
+    a.ungated = int(ungated); a.weight_in = int(on_input)
     a.idx = idx.data_ptr(); a.weight = weight.data_ptr(); a.act = act.data_ptr()
     a.shared = shared.data_ptr() if shared is not None else None
     a.shared_splits = shared.shape[0] if shared is not None else 0

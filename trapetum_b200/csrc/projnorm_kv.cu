@@ -8,7 +8,7 @@
 //   q <- q / sqrt(mean(q^2) + eps) * wq          mean over all H x dim numbers; wq of that size   (if wq is given)
 //   k <- k / sqrt(mean(k^2) + eps) * wk          mean over all G x dim numbers                    (if wk is given)
 //   q_h <- q_h * head_scale[h]                   (if given; the score is linear in q, so this weighs head h's scores)
-//   the first R dims of every q and k head turned by pos * inv_freq[i], pair (i, i + R/2)         (if R > 0)
+//   the first R dims of every q and k head turned by pos * inv_freq[i], pair (i, i + R/2), cos and sin times rot_mult   (if R > 0)
 //   gate_out[t][h] = sigmoid(gate column h)      (if asked for)
 //
 // The output row is [q heads | k heads | v heads], every head padded with zeros to D numbers (D >= dim, vdim: one
@@ -51,6 +51,7 @@ struct ProjNormKvArgs {
     int head_norm;                                // the norms are per head; their weights have dim numbers
     const float* v_first; float v_lam;            // [tokens][G * vdim] or null
     float* v_keep;                                // [tokens][G * vdim] or null
+    float rot_mult;                               // multiplies cos and sin
 };
 
 // The argument block's size, for the Python mirror's check.
@@ -145,7 +146,11 @@ __global__ void __launch_bounds__(1024) projnorm_kv_kernel(ProjNormKvArgs a) {
         }
     }
     // the angles of this token's position: once per token, not once per head
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf((float)pos * a.inv_freq[i], &sn[i], &cs[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+        float s_, c_;
+        sincosf((float)pos * a.inv_freq[i], &s_, &c_);
+        sn[i] = a.rot_mult * s_; cs[i] = a.rot_mult * c_;
+    }
     // where this token's k and v go in the cache (if anywhere); these dependent loads follow the row's, whose wait
     // has covered the position's and the sequence's
     bool store = false;

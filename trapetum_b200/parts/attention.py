@@ -54,11 +54,12 @@ Three more options change who sees whom and how the scores become weights; they 
 
 * ``block`` B (instead of ``window``): the query at position i sees key j iff ``j <= i`` and both lie in the same
   block of B positions, blocks counted from position 0 of the sequence; the cache line is a ring of B rows;
-* ``unit_sink``: the softmax denominator also holds ``exp(0)``, a sink without a key and without a value;
+* ``unit_sink``: the softmax denominator also holds ``exp(0)``, a sink without a key and without a value (without ``block``
+  and ``talk`` it is a ``sink`` of 0 for every head, below, and runs on the same kernels as that);
 * ``talk`` (a tensor name, [heads, heads]): the heads' scores are mixed before the mask and the softmax,
   ``s_h <- sum_g talk[h, g] s_g``.  Scale and ``head_temp`` are folded into the matrix when the weights are bound.
 
-Five more options of the same path, which go without ``proj_norm``, ``head_temp``, ``out_gate`` and the three above:
+Five more options of the same path, which go without ``block`` and ``talk`` (and ``head_norm`` without ``proj_norm``):
 
 * ``head_norm`` ``{"q": name, "k": name, "eps": e}``: every query / key head is divided by its root mean square over
   ``head_dim`` and multiplied by a weight of that size that the heads share, before the rotation (32-bit, inside
@@ -137,7 +138,7 @@ class Attention(Mixer):
         self.block = int(p["block"]) if p.get("block") else None
         self.unit_sink = bool(p.get("unit_sink"))
         self.talk_name = p.get("talk")
-        self.mixed = bool(self.block or self.unit_sink or self.talk_name)
+        self.mixed = bool(self.block or self.talk_name)
         if self.block and self.window:
             raise ValueError("attention: 'block' and 'window' exclude each other")
         if self.block is not None and self.block < 1:
@@ -148,13 +149,16 @@ class Attention(Mixer):
         self.v_mix = dict(p.get("v_mix") or {})
         self.value_gate_name = p.get("value_gate")
         per_head = bool(self.head_norm_names or self.sink_name or self.v_mix or self.value_gate_name)
-        if per_head and (self.proj_norm_names or self.head_temp_name or self.out_gate_name or self.mixed):
-            raise ValueError("attention: 'head_norm', 'sink', 'v_mix' and 'value_gate' go without 'proj_norm', 'head_temp', "
-                             "'out_gate', 'block', 'unit_sink' and 'talk'")
+        if per_head and self.mixed:
+            raise ValueError("attention: 'head_norm', 'sink', 'v_mix' and 'value_gate' go without 'block' and 'talk'")
+        if self.head_norm_names and self.proj_norm_names:
+            raise ValueError("attention: 'head_norm' and 'proj_norm' exclude each other")
+        if self.sink_name and self.unit_sink:
+            raise ValueError("attention: 'sink' and 'unit_sink' exclude each other")
         if self.head_norm_names:
             self.proj_norm_eps = float(hn.get("eps", 0.0))
         self.projected = bool(self.proj_norm_names or self.head_temp_name or self.out_gate_name or self.vd != self.hd
-                              or self.mixed or per_head)
+                              or self.mixed or self.unit_sink or per_head or self.position.amplitude != 1.0)
         self.order = self.position.head_order()
         if self.order is not None and (self.q_norm or self.k_norm):
             raise ValueError("attention: 'q_norm' and 'k_norm' go with a rotation of halves; use 'head_norm'")
@@ -234,6 +238,8 @@ class Attention(Mixer):
                 self.wk_norm = ordered(tensors[self.prefix + norms["k"]].float()).contiguous()
             if self.sink_name:
                 self.sink = tensors[self.prefix + self.sink_name].float().contiguous()
+            elif self.unit_sink and not self.mixed:
+                self.sink = torch.zeros(self.n_heads, dtype=torch.float32, device=q.device)      # exp(0) = 1
             if self.v_mix and not self.v_mix.get("first"):
                 self.v_lam = float(tensors[self.prefix + self.v_mix["weight"]].float())
             if self.head_temp_name:
@@ -449,7 +455,8 @@ class Attention(Mixer):
         qkv, gate = ops.projnorm_kv(part, H, G, self.hd, self.vd, D, dt, self.wq_norm, self.wk_norm, self.proj_norm_eps,
                                     None if self.mixed else self.head_temp, rotary, inv_freq, bool(self.out_gate_name),
                                     ctx.positions, ctx.token_seq, ctx.len_after, line.k, line.v, line.page_table,
-                                    line.ring_rows, self.b_proj, bool(self.head_norm_names), first, self.v_lam, keep)
+                                    line.ring_rows, self.b_proj, bool(self.head_norm_names), first, self.v_lam, keep,
+                                    self.position.amplitude)
         q = qkv[:, :H * D]
         k = qkv[:, H * D:(H + G) * D]
         v = qkv[:, (H + G) * D:]

@@ -120,6 +120,8 @@ class Norm(Part):
 
 
 class PositionEncoding(Part):
+    amplitude = 1.0          # a rotation's factor on cos and sin, which the mixer's kernel has to apply
+
     def head_order(self):
         """None, or the order (a list of ``head_dim`` places) in which a mixer has to lay out every q and k head's
         numbers so that the rotation becomes the rotate-half one that the kernels apply: a rotation of other pairs is

@@ -6,6 +6,8 @@
     h += post_mixer_norm(mixer(pre_mixer_norm(h)))
     h += post_ffn_norm(feed_forward(pre_ffn_norm(h)))
 
+(the second line only if the layer has a feed-forward).
+
 ``pre_norm``: the common two-norm arrangement, branch outputs added as they are:
 
     h += mixer(pre_mixer_norm(h));  h += feed_forward(pre_ffn_norm(h))
@@ -71,22 +73,36 @@ class _NormedBlock(Block):
 
 
 def _with_idle(block, specs: Dict[str, TensorSpec]) -> Dict[str, TensorSpec]:
-    """``idle``: tensor name -> size of vectors that a file may carry for a layer without feed-forward (the norm that
-    nothing follows); they are accepted and not used."""
+    """``idle``: tensor name -> size (or shape) of tensors that a file may carry for a layer without feed-forward (the norm
+    that nothing follows); they are accepted and not used."""
     for name, size in (block.params.get("idle") or {}).items():
-        specs.setdefault(block.prefix + name, TensorSpec((int(size),), "norm", optional=True))
+        shape = tuple(size) if isinstance(size, (list, tuple)) else (int(size),)
+        specs.setdefault(block.prefix + name, TensorSpec(shape, "norm", optional=True))
     return specs
 
 
 class SandwichBlock(_NormedBlock):
+    """``pre_ffn_norm`` and ``post_ffn_norm`` may be None for a layer whose feed-forward is of kind "none"; ``idle``: see
+    :class:`PreNormBlock`."""
     NORMS = ("pre_mixer_norm", "post_mixer_norm", "pre_ffn_norm", "post_ffn_norm")
+
+    def __init__(self, params, prefix, rt, mixer, feed_forward):
+        Block.__init__(self, params, prefix, rt, mixer, feed_forward)
+        self.has_ffn = not getattr(feed_forward, "absent", False)
+        if self.has_ffn and not (params.get("pre_ffn_norm") and params.get("post_ffn_norm")):
+            raise ValueError("sandwich: a layer with a feed-forward needs 'pre_ffn_norm' and 'post_ffn_norm'")
+        self.norms = {n: build_part("norm", params[n], prefix, rt) for n in self.NORMS if self.has_ffn or "mixer" in n}
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return _with_idle(self, super().tensor_specs())
 
     def forward(self, stream, ctx, cache) -> None:
         dt = self.rt.dtype
         x = stream.normed(self.norms["pre_mixer_norm"], dt)
         stream.add_normed(self.mixer.forward(x, ctx, cache), self.norms["post_mixer_norm"])
-        x = stream.normed(self.norms["pre_ffn_norm"], dt)
-        stream.add_normed(self.feed_forward.forward(x, ctx), self.norms["post_ffn_norm"])
+        if self.has_ffn:
+            x = stream.normed(self.norms["pre_ffn_norm"], dt)
+            stream.add_normed(self.feed_forward.forward(x, ctx), self.norms["post_ffn_norm"])
 
 
 class PreNormBlock(_NormedBlock):

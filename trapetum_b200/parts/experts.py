@@ -13,7 +13,9 @@ False makes the experts ``down_e(act(up_e x))`` with a unary activation ("relu2"
 matrix; the shared expert is then of that form too.  ``route_scale`` multiplies the winners' weights.
 ``router_bias`` (a tensor name, one number per expert) is added to the logits themselves, by the routing kernel.  A softmax over the
 winners' logits only is ``score`` "softmax" with ``weight_eps`` 0: the winners' shares of the softmax over all
-experts, divided by their sum, are exactly that.
+experts, divided by their sum, are exactly that.  ``renormalize`` False takes the winners' scores as the weights, undivided.
+``weight_on`` "input": the weight multiplies what the expert reads, ``down_e(act(gate_e (w x)) * up_e (w x))``, and the
+output is the plain sum of the winners' outputs.
 
 Parameters (none is fixed in code): ``hidden_size``, ``experts``, ``top``, ``intermediate_size``, ``activation``
 ("silu"), ``score`` ("sigmoid"), ``groups``, ``keep_groups``, ``group_score_of``, ``weight_eps``, the tensor names
@@ -56,6 +58,10 @@ class RoutedExperts(FeedForward):
         self.activation = p.get("activation", "silu")
         self.score = p.get("score", "sigmoid")
         self.route_scale = float(p.get("route_scale", 1.0))
+        self.renormalize = bool(p.get("renormalize", True))
+        self.weight_on = p.get("weight_on", "output")
+        if self.weight_on not in ("input", "output"):
+            raise ValueError(f"routed_experts: weight_on '{self.weight_on}' (known: input, output)")
         if self.activation != ("silu" if self.gated else "relu2") or self.score not in ("sigmoid", "softmax"):
             raise ValueError("routed_experts: the kernels know gated experts with silu, ungated experts with relu2, and "
                              "sigmoid or softmax scores")
@@ -141,7 +147,7 @@ class RoutedExperts(FeedForward):
         logits = linear_partials(x, self.w_router_up if fused_up else self.w_router)
         idx, weight, gate = ops.moe_route(logits, self.E, self.correction, self.has_gate, self.top, self.groups,
                                           self.keep, self.group_top, self.weight_eps, self.score, self.route_scale,
-                                          self.router_bias)
+                                          self.router_bias, self.renormalize)
         shared = None
         if self.shared is not None:
             # float32 partial sums [splits, T, hidden]
@@ -152,7 +158,7 @@ class RoutedExperts(FeedForward):
                 if not self._ones or self._ones[-1].numel() < x.shape[0]:
                     self._ones.append(torch.ones(max(256, 2 * x.shape[0]), dtype=torch.float32, device=x.device))
                 gate = self._ones[-1]
-        return ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, idx, weight, shared, gate, self.w_gate_up)
+        return ops.moe_experts(x, self.w_gate, self.w_up, self.w_down, idx, weight, shared, gate, self.w_gate_up, self.weight_on)
 
 
 register_part("feed_forward", "routed_experts", RoutedExperts)

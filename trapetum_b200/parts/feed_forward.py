@@ -8,7 +8,7 @@ activation ``clamped_swish`` takes a ``limit`` L and bounds both branches:
 ``g' = min(g, L)``, ``u' = clamp(u, -L, L)``, ``g' sigmoid(1.702 g') (u' + 1)``.
 
 ``mlp`` is the form without a gate branch, ``down(act(up(x)))``, with a unary
-activation (``relu2``: the square of relu).
+activation (``relu2``: the square of relu; ``gelu``: the exact one, ``u Phi(u)``).
 
 Also here: ``none`` (a layer without a feed-forward) and ``token_gated``, a narrow
 side input that is looked up by token id:
@@ -79,7 +79,7 @@ class GatedMLP(FeedForward):
 
 
 class PlainMLP(FeedForward):
-    """``down(act(up(x)))``.  Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (a unary one: "relu2")
+    """``down(act(up(x)))``.  Parameters: ``hidden_size``, ``intermediate_size``, ``activation`` (a unary one: "relu2", "gelu")
     and the tensor names ``up`` and ``down``.  With many tokens the activation runs in the tensor-core product's
     epilogue; with few, the product keeps its split-K partial sums and a small kernel adds and activates them."""
     graph_safe = True          # every launch depends on device data only

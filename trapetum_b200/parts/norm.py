@@ -118,5 +118,47 @@ class LayerNorm(Norm):
         return ops.add_layernorm(h, a, self.weight, self.bias, self.eps, out_dtype)
 
 
+class DynamicTanh(Norm):
+    """``y = tanh(alpha * x) * w + b``: no statistics, so no number of a row waits for any other.  ``alpha`` is one number
+    (stored as a tensor without axes), ``w`` and ``b`` vectors; all of it 32-bit.  Parameters: ``size`` and the tensor
+    names ``weight``, ``bias`` and ``alpha``.  The residual sum before it, with or without a norm of this kind on the
+    branch, runs in the same kernel (``ops.dyt``)."""
+
+    def __init__(self, params, prefix, rt):
+        super().__init__(params, prefix, rt)
+        self.size = int(params["size"])
+        self.norm = None             # (alpha, weight, bias) as ops.dyt takes it
+
+    def tensor_specs(self) -> Dict[str, TensorSpec]:
+        return {self._name("weight"): TensorSpec((self.size,), "gain"), self._name("bias"): TensorSpec((self.size,), "norm"),
+                self._name("alpha"): TensorSpec((), "gain")}
+
+    def bind(self, tensors) -> None:
+        # they enter 32-bit arithmetic: kept in 32 bits (exact for what a file stores in 16)
+        self.norm = (float(tensors[self._name("alpha")].float()), tensors[self._name("weight")].float().contiguous(),
+                     tensors[self._name("bias")].float().contiguous())
+
+    def kernel_files(self):
+        return ("dyt",)
+
+    def apply(self, x: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+        return ops.dyt(None, x, norm_b=self.norm, out_dtype=out_dtype)
+
+    def add_to(self, h, a, then, out_dtype):
+        if then is None or isinstance(then, DynamicTanh):
+            return ops.dyt(h, a, self.norm, None if then is None else then.norm, out_dtype)
+        ops.dyt(h, a, self.norm)
+        return then.apply(h, out_dtype)
+
+    def add_copy(self, h: torch.Tensor, a: torch.Tensor, out: torch.Tensor) -> None:
+        """``h += self(a)`` in place, and the new ``h`` rounded into ``out`` (rows of any stride); one kernel."""
+        ops.dyt(h, a, self.norm, out=out)
+
+    def set_apply(self, h: torch.Tensor, a: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+        """``h <- a`` in place (a product, or its split-K partial sums, that replaces the stream), returns ``norm(h)``."""
+        return ops.dyt(h, a, None, self.norm, out_dtype, replace=True)
+
+
 register_part("norm", "rmsnorm", RMSNorm)
+register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "layernorm", LayerNorm)

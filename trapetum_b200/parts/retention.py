@@ -47,6 +47,8 @@ class Retention(Mixer):
         self.position = build_part("position", p["position"], prefix, rt)
         if self.position.rotary_table() is None:
             raise ValueError("retention: 'position' must be a rotation or none")
+        if self.position.amplitude != 1.0:
+            raise ValueError("retention: a rotation with a factor on cos and sin is not built")
 
     def tensor_specs(self) -> Dict[str, TensorSpec]:
         HD, HV = self.heads * self.D, self.heads * self.V

@@ -12,6 +12,10 @@ matrix and its cache line in one call.
 ``pairing`` "neighbours" is the interleaved layout, pairs ``(x[2i], x[2i+1])``: a mixer that lays out its q and k
 heads in :meth:`Rope.head_order` (even places of the rotated part first) runs it as the rotate-half rotation.
 ``table`` "float64" makes the frequencies in 64-bit before they are stored in 32.
+
+``scaling`` (instead of ``scaling_factor``): a dict as :func:`rotary_frequencies` takes it, for instance a blend per
+frequency between the plain and the scaled one.  It may come with a factor on cos and sin (:attr:`Rope.amplitude`),
+which a mixer has to hand to its kernel; a mixer that cannot refuses the encoding.
 """
 from __future__ import annotations
 
@@ -62,6 +66,9 @@ class Rope(PositionEncoding):
             raise ValueError(f"rope: rotary_dim {self.rotary_dim} must be even and within head_dim {self.head_dim}")
         idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32)
         self.scaling_factor = float(params.get("scaling_factor") or 1.0)
+        scaling = dict(params.get("scaling") or {})
+        if scaling and self.scaling_factor != 1.0:
+            raise ValueError("rope: 'scaling' and 'scaling_factor' exclude each other")
         if not self.scaling_factor > 0.0:
             raise ValueError(f"rope: scaling_factor must be positive, got {self.scaling_factor}")
         self._inv_freq_cpu = 1.0 / (torch.tensor(self.theta, dtype=torch.float32) ** (idx / self.rotary_dim))
@@ -70,6 +77,8 @@ class Rope(PositionEncoding):
         if params.get("table", "float32") == "float64":
             self._inv_freq_cpu, _ = rotary_frequencies(self.rotary_dim, self.theta,
                                                        {"factor": self.scaling_factor} if self.scaling_factor != 1.0 else None)
+        if scaling:
+            self._inv_freq_cpu, self.amplitude = rotary_frequencies(self.rotary_dim, self.theta, scaling)
         self.pairing = params.get("pairing", "halves")
         if self.pairing not in ("halves", "neighbours"):
             raise ValueError(f"rope: pairing '{self.pairing}' (known: halves, neighbours)")
@@ -94,6 +103,8 @@ class Rope(PositionEncoding):
         """Rotate q and k inside ``qkv`` at the step's positions; with ``store`` also
         write k and v into the cache line.  ``partial``: split-K partial sums of the projection
         ([splits, tokens, width] float32) to take the values from; ``qkv`` is then only written."""
+        if self.amplitude != 1.0:
+            raise NotImplementedError("rope: this kernel has no factor on cos and sin")
         ops.rope_kv(qkv, n_heads, n_kv_heads, self.head_dim, self.rotary_dim, self.inv_freq,
                     ctx.positions, ctx.token_seq, ctx.len_after,
                     line.k if store else None, line.v if store else None,

@@ -11,6 +11,9 @@ Arrangements that norm AFTER the sum replace the stream instead of adding to it:
 :meth:`fold_normed` is ``h <- norm(alpha * h + a)``, and their sublayers read the
 stream itself through :meth:`read` (a copy in the compute dtype when that is not
 32-bit), which rides along with whatever was still waiting.
+
+:meth:`copy_into` writes the stream, rounded, into part of a wider matrix (a product that reads the stream beside
+something else), and :meth:`replace` makes a product the new stream.
 """
 from __future__ import annotations
 
@@ -53,12 +56,40 @@ class ResidualStream:
         self._flush()
         self._pending = (a, norm, float(alpha))
 
+    def replace(self, a: torch.Tensor) -> None:
+        """h <- a (float32 [tokens, hidden], or [splits, tokens, hidden] partial sums); whatever was waiting must have been
+        applied before ``a`` was made, so nothing may be waiting now."""
+        if self._pending is not None:
+            raise RuntimeError("residual stream: an addition is still waiting; the product that replaces the stream has not seen it")
+        if a.dim() == 3 and a.shape[0] == 1:
+            a = a[0]
+        if a.dim() == 2:
+            self.h = a                     # the product's own memory becomes the stream
+        else:
+            self._pending = (a, None, ("set",))
+
+    def copy_into(self, out: torch.Tensor) -> None:
+        """The stream, after whatever addition was still waiting, rounded to ``out``'s dtype into ``out`` [tokens, hidden],
+        whose rows may be parts of wider ones; one kernel where the waiting norm offers it."""
+        if self._pending is not None and self._pending[1] is not None and self._pending[2] is None \
+                and hasattr(self._pending[1], "add_copy"):
+            a, post, _ = self._pending
+            self._pending = None
+            post.add_copy(self.h, a, out)
+            return
+        self._flush()
+        ops.dyt(self.h, out=out)
+
     def normed(self, norm: Norm, out_dtype: torch.dtype) -> torch.Tensor:
         """norm(h), after whatever addition was still waiting."""
         if self._pending is not None and self._pending[2] == ("terms",) and hasattr(norm, "add_terms_apply"):
             terms = self._pending[0]
             self._pending = None
             return norm.add_terms_apply(self.h, terms, out_dtype)[0]      # the sum of the terms and the norm in one kernel
+        if self._pending is not None and self._pending[2] == ("set",) and hasattr(norm, "set_apply"):
+            a = self._pending[0]
+            self._pending = None
+            return norm.set_apply(self.h, a, out_dtype)      # the partial sums' sum and the norm in one kernel
         if self._pending is not None and isinstance(self._pending[2], tuple) and self._pending[2][0] == "scaled":
             branches, _, (_, scale) = self._pending
             if hasattr(norm, "add_scaled_apply"):
@@ -115,7 +146,9 @@ class ResidualStream:
             return
         a, post, alpha = self._pending
         self._pending = None
-        if alpha == ("terms",):
+        if alpha == ("set",):
+            self.h = ops.sum_partials(a)
+        elif alpha == ("terms",):
             ops.add_terms_rmsnorm(self.h, a)
         elif isinstance(alpha, tuple):
             ops.add_scaled_rmsnorm(self.h, a, alpha[1])
