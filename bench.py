@@ -23,6 +23,7 @@ MEASURED_PEAKS.json beside this file when the driver wrote it, otherwise from th
     python bench.py --design fidepel [--sizes small,medium,large] [--batch 8] [--context 2048]
     python bench.py --design fibelix [--sizes small,medium,large] [--batch 8] [--context 2048]
     python bench.py --design ranilix [--sizes small,medium,large] [--batch 8] [--context 2048]
+    python bench.py --design sezanex [--sizes small,medium,large] [--batch 8] [--context 2048]
 
 ``--design divanex`` is a measurement of its own (the default workload and its line stay as they are): Divanex
 models with random weights at a few layer sizes, a 2,048-token prompt and decode steps of ``batch`` sequences
@@ -1221,6 +1222,234 @@ def ranilix_compare(args, torch):
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------------------
+# --design sezanex: the design at sizes that resemble real layers, beside Divanex (the closest model of the library:
+# attention and Mamba-2 layers in turn, on the same host) with as many layer calls, at equal width, head counts, head
+# sizes, state and vocabulary
+# ---------------------------------------------------------------------------------------------------------------
+# name -> (window; experts, winners, an expert's inner width); the rest are DESIGN_SIZES'
+SEZANEX_SIZES = {"small": (1024, 16, 2, 512), "medium": (1024, 32, 2, 1024), "large": (1024, 32, 2, 1792)}
+
+
+def sezanex_config(size):
+    """Three quarters of DESIGN_SIZES' layers, of which a third runs twice: as many calls as that size has layers."""
+    W, L, H, G, d, ff, mh, mp, N, V = DESIGN_SIZES[size]
+    win, E, top, eff = SEZANEX_SIZES[size]
+    attn = {"type": "attention", "mixer": {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "mask": {"size": win},
+                                           "rot": {"dims": d, "base": 500000.0, "scaling": {"factor": 8.0, "original": 8192,
+                                                                                            "fast": 32.0, "slow": 1.0}}},
+            "mlp": {"kind": "dense", "ff": ff}}
+    ssm = {"type": "mamba2", "mixer": {"heads": mh, "vdim": mp, "state": N, "groups": 2, "conv": 4, "norm_groups": 2},
+           "mlp": {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}}}
+    n = 3 * L // 4
+    return {"architecture": "Sezanex", "vocab": V, "width": W, "norm": {"eps": 1e-6},
+            "layers": [attn if i % 2 == 0 else ssm for i in range(n)],
+            "loop": {"start": L // 4, "stop": L // 2, "times": 2}}
+
+
+def sezanex_bytes_flops(cfg, tokens, ctx, batch):
+    """(weight bytes a decode step reads, cache and state bytes per sequence at ``ctx`` tokens, tensor-core FLOPs and
+    32-bit recurrence FLOPs of one ``tokens``-token prompt); a layer that runs twice is read and computed twice, and an
+    expert's matrices are read if one of ``batch`` tokens is expected to choose it."""
+    W, V = cfg["width"], cfg["vocab"]
+    wb, cb, fl, rf = V * W + 2 * W, 0, 2 * V * W, 0
+    lp = cfg["loop"]
+    for i, L in enumerate(cfg["layers"]):
+        times = lp["times"] if lp["start"] <= i < lp["stop"] else 1
+        if i == lp["start"]:
+            wb += times * 2 * W * W
+            fl += times * 4 * tokens * W * W
+        m, ml = L["mixer"], L["mlp"]
+        read = used = 8 * W
+        if L["type"] == "attention":
+            H, G, D, Vd = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            span = min(tokens, m["mask"]["size"])
+            mats = (H * D + G * (D + Vd)) * W + W * H * Vd
+            cb += times * G * (D + Vd) * min(ctx, m["mask"]["size"]) * 2
+            fl += times * 2 * H * (D + Vd) * (span * (span + 1) // 2 + (tokens - span) * span)
+        else:
+            inner = m["heads"] * m["vdim"]
+            ch = inner + 2 * m["groups"] * m["state"]
+            mats = (inner + ch + m["heads"]) * W + W * inner + ch * m["conv"]
+            cb += times * 2 * 4 * (inner * m["state"] + (m["conv"] - 1) * ch)      # the state is read and written, 32-bit
+            rf += times * tokens * inner * m["state"] * 5
+        read, used = read + mats, used + mats
+        if ml["kind"] == "dense":
+            read, used = read + 2 * ml["ff"] * W, used + 2 * ml["ff"] * W
+        else:
+            E, top, per = ml["router"]["experts"], ml["router"]["top"], 3 * ml["expert"]["ff"] * W
+            read += E * W + per * E * (1.0 - (1.0 - top / E) ** batch)
+            used += E * W + per * top
+        wb += times * read
+        fl += times * 2 * tokens * used
+    return int(2 * wb), cb, fl, rf
+
+
+def sezanex_kernels(torch, size, hbm_gbs, tokens=PREFILL_TOKENS):
+    """The design's own kernels alone, each beside the like kernel of the library's other models: microseconds, algorithmic
+    bytes (or FLOPs) and the fraction of the roofline.  One prompt of ``tokens`` tokens; 64 sequences at 2,048 for the
+    one-token kernels."""
+    from trapetum_b200.csrc import ops
+    W, _, H, G, d, ff, mh, mp, N, _ = DESIGN_SIZES[size]
+    win, E, top, eff = SEZANEX_SIZES[size]
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    T, B, ctx = tokens, 64, 2048
+    out = {}
+    tc_peak = peaks()[1]
+
+    def rec(name, us, nbytes, like=None, tensor_flops=0.0, fp32_flops=0.0):
+        t_mem, t_tc = nbytes / (hbm_gbs * 1e9) * 1e6, tensor_flops / (tc_peak * 1e12) * 1e6
+        t_fma = fp32_flops / (FP32_TFLOPS_NOMINAL * 1e12) * 1e6
+        best = max(t_mem, t_tc, t_fma)
+        out[name] = {"us": round(us, 1), "bytes": int(nbytes), "roofline_us": round(best, 1), "frac": round(best / us, 3),
+                     "bound": "tensor" if best == t_tc else ("fp32" if best == t_fma else "hbm")}
+        if like:
+            out[name]["like"] = like
+    f32 = lambda *s: torch.randn(*s, device=dev)
+    rb = lambda *s: (torch.randn(*s, device=dev) * 0.5).to(bf)
+    one = ", one token for each of 64 sequences"
+    pos, tseq = torch.arange(T, device=dev).int(), torch.zeros(T, device=dev).int()
+    ss, la = torch.tensor([0, T], device=dev).int(), torch.tensor([T], device=dev).int()
+    slot0 = torch.zeros(1, device=dev).int()
+    pos1 = torch.full((B,), ctx - 1, device=dev).int()
+    ss1, tseq1, la1 = torch.arange(B + 1, device=dev).int(), torch.arange(B, device=dev).int(), torch.full((B,), ctx, device=dev).int()
+    # ---- the residual sum with the norms around it, and the stream beside the embedding
+    wbf = torch.ones(W, device=dev).to(bf)
+    na, nb_ = ((0.7, torch.ones(W, device=dev), torch.zeros(W, device=dev)) for _ in range(2))
+    for what, TT, splits in (("", T, 1), (one, B, 4)):
+        h, a = f32(TT, W), f32(splits, TT, W)
+        both = torch.empty(TT, 2 * W, dtype=bf, device=dev)
+        nbytes = TT * W * (8 + 4 * splits + 2)
+        rec("dyt (sum and two norms)" + what, _median_us(torch, lambda: ops.dyt(h, a, na, nb_, bf), flush), nbytes, like="add_rmsnorm" + what)
+        rec("dyt (sum, norm and copy)" + what, _median_us(torch, lambda: ops.dyt(h, a, na, out=both[:, :W]), flush), nbytes, like="add_rmsnorm" + what)
+        rec("add_rmsnorm" + what, _median_us(torch, lambda: ops.add_rmsnorm(h, a, wbf, 1e-5, 0.0, wbf, 1e-5, 0.0, bf), flush), nbytes)
+    # ---- between the attention's products and its kernel
+    pages = (T + 63) // 64
+    inv = torch.rand(d // 2, device=dev)
+    wide = (H * d + 2 * G * d + 15) // 16 * 16
+    wq, wk = torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+    for what, TT, po, ts, le, splits in (("", T, pos, tseq, la, 1), (one, B, pos1, tseq1, la1, 4)):
+        part = f32(splits, TT, wide)
+        n_seq = le.numel()
+        kp, vp = (torch.zeros(n_seq * pages, G, 64, d, dtype=bf, device=dev) for _ in range(2))
+        table = torch.arange(n_seq * pages, device=dev).int().view(n_seq, pages)
+        nb = TT * 2 * G * d * 2
+        rec("projnorm_kv (rotation with a factor)" + what,
+            _median_us(torch, lambda: ops.projnorm_kv(part, H, G, d, d, d, bf, wq, wk, 1e-6, None, d, inv, False, po, ts, le, kp, vp, table, 0, rot_mult=1.2), flush),
+            nb + TT * (H + 2 * G) * d * (4 * splits + 2), like="headnorm_kv" + what)
+        hpart = f32(splits, TT, (H + G) * d)
+        rec("headnorm_kv" + what,
+            _median_us(torch, lambda: ops.headnorm_kv(hpart, H, G, d, bf, True, True, True, 1e-5, 0.5, 64, po, ts, le, kp, vp, table, 0), flush),
+            nb + TT * ((H + G) * 4 * splits + (H + 2 * G) * 2) * d)
+    # ---- attention with a unit sink and a window, beside the same kernel without a sink
+    q, k, v, sink = rb(T, H * d), rb(T, G * d), rb(T, G * d), torch.zeros(H, device=dev)
+    n_pairs = win * (win + 1) // 2 + (T - win) * win
+    nb = (2 * H + 2 * G) * d * T * 2
+    rec("attention with a sink (prefill)", _median_us(torch, lambda: ops.attn_prefill_sink(q, k, v, ss, tseq, H, d, d ** -0.5, sink, T, [T], win, n_kv_heads=G), flush),
+        nb, like="attention (prefill)", tensor_flops=4.0 * H * d * n_pairs)
+    rec("attention (prefill)", _median_us(torch, lambda: ops.attn_prefill(q, k, v, ss, tseq, H, G, d, d ** -0.5, 0.0, win, T, [T]), flush),
+        nb, tensor_flops=4.0 * H * d * n_pairs)
+    kp, vp = rb(B * win // 64, G, 64, d), rb(B * win // 64, G, 64, d)
+    tab, q1 = torch.arange(B * win // 64, device=dev).int().view(B, win // 64), rb(B, H * d)
+    for name, s in (("attention with a sink (decode)", sink), ("attention (decode)", None)):
+        rec(name, _median_us(torch, lambda: ops.attn_decode(q1, kp, vp, tab, la1, H, G, d, d ** -0.5, 0.0, win, win, ctx, sink=s), flush),
+            B * 2 * G * d * win * 2, like="attention (decode)" if s is not None else None)
+    # ---- the state-space mixer with two groups, beside one group
+    for groups in (2, 1):
+        inner, ch = mh * mp, mh * mp + 2 * groups * N
+        cw, cb, dtb, Al, D, nw = f32(ch, 4) * .3, f32(ch) * .1, f32(mh) - 1, f32(mh) * .5, f32(mh), f32(inner)
+        st, st64 = (torch.zeros(n, ops.mamba2_state_size(mh, mp, N, groups, 4), device=dev) for n in (1, B))
+        proj, dtr, proj1, dtr1 = rb(T, inner + ch), f32(T, mh), rb(B, inner + ch), f32(B, mh)
+        name = f"mamba2, {groups} group{'s' * (groups > 1)}"
+        like = "mamba2, 1 group" if groups > 1 else None
+        rec(name, _median_us(torch, lambda: ops.mamba2(proj, dtr, mh, mp, N, groups, 4, groups, cw, cb, dtb, Al, D, nw, 1e-5, st, ss, tseq, slot0, 1, False,
+                                                       max_seq_len=T), flush),
+            T * (ch * 2 * 3 + inner * 2 + inner * 4 * 2 + inner * 2), fp32_flops=T * inner * N * 5.0, like=like)
+        rec(name + one, _median_us(torch, lambda: ops.mamba2(proj1, dtr1, mh, mp, N, groups, 4, groups, cw, cb, dtb, Al, D, nw, 1e-5, st64, ss1, tseq1, tseq1, B, True), flush),
+            st64.numel() * 8, like=like + one if like else None)
+    # ---- the dense feed-forward's first product with the exact gelu, beside the square of relu
+    x, x1 = rb(T, W), rb(B, W)
+    wup = rb(ff, W) * .02
+    for act in ("gelu", "relu2"):
+        like = "relu2" if act == "gelu" else None
+        rec(f"up product with {act}", _median_us(torch, lambda: ops.gemm_tc(x, wup, bf, unary_act=act), flush), 2 * (ff * W + T * W + T * ff),
+            tensor_flops=2.0 * T * ff * W, like=like and f"up product with {like}")
+        up1 = f32(4, B, ff)
+        rec(f"{act} of partial sums" + one, _median_us(torch, lambda: ops.unary_act(up1, act, bf), flush), B * ff * (16 + 2),
+            like=like and f"{like} of partial sums" + one)
+    # ---- the experts: weights on what they read, beside weights on what they return
+    gw, uw, dw = rb(E, eff, W) * .02, rb(E, eff, W) * .02, rb(E, W, eff) * .02
+    gu = torch.stack([ops.interleave_gate_up(gw[e], uw[e]) for e in range(E)]).contiguous()      # as the part binds them
+    for what, xx in (("", x), (one, x1)):
+        TT = xx.shape[0]
+        lg = f32(1, TT, (E + 15) // 16 * 16)
+        for raw in (True, False):
+            name = "moe_route (scores as weights)" if raw else "moe_route (shares as weights)"
+            rec(name + what, _median_us(torch, lambda: ops.moe_route(lg, E, None, False, top, 1, 1, 1, 1e-20, renormalize=not raw), flush),
+                lg.numel() * 4 + TT * top * 8, like="moe_route (shares as weights)" + what if raw else None)
+        idx, wt, _ = ops.moe_route(lg, E, None, False, top, 1, 1, 1, 0.0, renormalize=False)
+        n_used = int(torch.unique(idx).numel())
+        for on in ("input", "output"):
+            rec(f"experts (weight on the {on})" + what, _median_us(torch, lambda: ops.moe_experts(xx, gw, uw, dw, idx, wt, gate_up_w=gu, weight_on=on), flush),
+                3 * n_used * eff * W * 2 + TT * W * (2 + 4), tensor_flops=2.0 * TT * top * 3 * eff * W,
+                like="experts (weight on the output)" + what if on == "input" else None)
+    # ---- the product that replaces the stream
+    both, win_w = rb(T, 2 * W), rb(W, 2 * W) * .02
+    rec("loop.in product", _median_us(torch, lambda: ops.gemm_tc(both, win_w, torch.float32, partials=True), flush), 2 * (2 * W * W + 2 * T * W) + 4 * T * W,
+        tensor_flops=4.0 * T * W * W, like="up product with relu2")
+    return out
+
+
+def sezanex_compare(args, torch):
+    """Prints one JSON line: per size, Sezanex and the Divanex model of as many layer calls and equal width, heads, state and
+    vocabulary (prefill of one 2,048-token prompt, decode at ``batch`` x ``context``), with bytes, FLOPs and roofline
+    fractions, and the design's kernels alone beside their like kernels."""
+    import trapetum_b200 as tb
+    from trapetum_b200.csrc import ops
+    hbm_gbs, bf16_tflops, peak_src = peaks()
+    warmup = max(3, args.warmup)
+    ctx, batch = args.context, args.batch
+    out = {"design": "sezanex", "beside": "divanex", "sizes": {},
+           "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": bf16_tflops, "source": peak_src, "fp32_tflops_nominal": FP32_TFLOPS_NOMINAL},
+           "dtype": "bf16", "data": "synthetic (random weights, random token ids)", "batch": batch, "context": ctx,
+           "timing": "CUDA events; decode: median of five regions of --steps steps; kernels alone: a 256 MB buffer is written "
+                     "between timed launches (larger than L2)"}
+    clocks = ClockSampler()
+    clocks.__enter__()
+    for size in [s for s in args.sizes.split(",") if s in DESIGN_SIZES]:
+        row = {}
+        for which in ("sezanex", "divanex"):
+            cfg = sezanex_config(size) if which == "sezanex" else divanex_config(size)
+            V = cfg["vocab"]
+            model = tb.random_model(cfg, 7, 0.02, 0.1, "bfloat16", "cuda:0", host="python")
+            engine = tb.Engine(model, max_tokens=batch * (ctx + 64), max_slots=batch)
+            random_cache(engine)
+            pms, hms, _ = time_prefill(engine, torch, PREFILL_TOKENS, V, reps=5, warmup=warmup)
+            r = time_decode(engine, torch, [ctx] * batch, args.steps, warmup, V, clocks=clocks)
+            wb, cb, fl, rf = (sezanex_bytes_flops if which == "sezanex" else divanex_bytes_flops)(cfg, PREFILL_TOKENS, ctx, batch)
+            nbytes = wb + batch * cb
+            pre_ideal = fl / (bf16_tflops * 1e12) + rf / (FP32_TFLOPS_NOMINAL * 1e12)
+            row[which] = {
+                "prefill": {"tokens": PREFILL_TOKENS, "ms": round(pms, 3), "host_ms": round(hms, 3), "tok_s": round(PREFILL_TOKENS * 1e3 / pms, 1),
+                            "tensor_flops": fl, "fp32_recurrence_flops": rf, "frac_of_roofline": round(pre_ideal * 1e3 / pms, 4)},
+                "decode": {"ms": r["ms"], "tok_s": round(batch * 1e3 / r["ms"], 1), "bytes": nbytes,
+                           "gbs": round(nbytes / (r["ms"] * 1e-3) / 1e9, 1),
+                           "frac_of_hbm": round(nbytes / (r["ms"] * 1e-3) / 1e9 / hbm_gbs, 4), "launches": r["launches"]},
+            }
+            engine.check_kernels()
+            del engine, model
+            torch.cuda.empty_cache()
+        if not args.no_points:
+            row["kernels_alone"] = sezanex_kernels(torch, size, hbm_gbs)
+        out["sizes"][size] = row
+    clocks.__exit__()
+    out["clocks"] = clocks.summary()
+    out["kernel_errors"] = ops.kernel_errors()
+    print(json.dumps(out))
+    return 0
+
+
 HOST = None              # which host runs the models (None: the library's default, the native host for these models)
 
 
@@ -1569,9 +1798,10 @@ def main() -> int:
     ap.add_argument("--leave-out", action="store_true",
                     help="instead of the bench line: the decode step re-timed with one kind of launch left out at a "
                          "time (its results are then wrong; only its time is of interest), one line per kind")
-    ap.add_argument("--design", default=None, choices=["divanex", "lofirax", "fidepel", "fibelix", "ranilix"],
+    ap.add_argument("--design", default=None, choices=["divanex", "lofirax", "fidepel", "fibelix", "ranilix", "sezanex"],
                     help="instead of the bench line: this design at the layer sizes of --sizes beside the library's closest "
-                         "model at equal size (divanex beside Gemma-2, lofirax beside divanex, fidepel beside Gemma-2, fibelix beside fidepel)")
+                         "model at equal size (divanex beside Gemma-2, lofirax beside divanex, fidepel beside Gemma-2, fibelix beside fidepel, "
+                         "ranilix and sezanex beside divanex)")
     ap.add_argument("--sizes", default="small,medium,large", help="with --design: which of small, medium, large")
     ap.add_argument("--gemm-compare", type=int, default=0, metavar="TOKENS",
                     help="instead of the bench line: the four products of a layer of --model at TOKENS tokens, this "
@@ -1599,6 +1829,8 @@ def main() -> int:
             return fibelix_compare(args, torch)
         if args.design == "ranilix":
             return ranilix_compare(args, torch)
+        if args.design == "sezanex":
+            return sezanex_compare(args, torch)
         return lofirax_compare(args, torch) if args.design == "lofirax" else design_compare(args, torch)
     if args.gemm_compare:
         return gemm_compare(MODELS[args.model], torch, args.gemm_compare, peaks()[1])
