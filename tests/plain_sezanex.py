@@ -196,10 +196,16 @@ def dense(h, t, p, rnd=same):
     return rnd(gelu(h @ f64(t[p + "up"]).T)) @ f64(t[p + "down"]).T
 
 
+MARGINS = None                   # a list while routing margins are collected
+
+
 def route(h, router, top: int):
     """(winners [T, top], their scores [T, top])."""
-    s = torch.sigmoid(h @ router.T)
-    order = torch.sort(s, dim=-1, descending=True, stable=True)
+    z = h @ router.T
+    order = torch.sort(torch.sigmoid(z), dim=-1, descending=True, stable=True)
+    if MARGINS is not None and top < z.shape[1]:
+        ranked = torch.sort(z, dim=-1, descending=True).values
+        MARGINS.append(ranked[:, top - 1] - ranked[:, top])
     return order.indices[:, :top], order.values[:, :top]
 
 
@@ -282,6 +288,17 @@ def logits(cfg, tensors, tokens, pieces=None, rnd=same) -> torch.Tensor:
 
 def forward(cfg, tensors, tokens, rnd=same) -> torch.Tensor:
     return logits(cfg, tensors, tokens, None, rnd)
+
+
+def routing_margin(cfg, tensors, tokens) -> float:
+    """The smallest distance, in router logits, between a winner and a loser of any routing decision of the sequence."""
+    global MARGINS
+    MARGINS = []
+    try:
+        forward(cfg, tensors, tokens)
+        return min((float(m.min()) for m in MARGINS), default=float("inf"))
+    finally:
+        MARGINS = None
 
 
 def generate_greedy(cfg, tensors, prompt, n: int) -> List[int]:
