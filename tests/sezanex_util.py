@@ -104,7 +104,7 @@ def random_weights(cfg: dict, seed: int, sharp: float = 2.0) -> dict:
 
     E = torch.randn(V, W, generator=g)
     if C:
-        levels = torch.linspace(-1.6, 1.6, C) if C > 1 else torch.zeros(1)
+        levels = torch.atanh(0.8 - 0.1 * torch.arange(C)) / 0.72          # evenly spaced behind the norm's tanh
         E[:, :C] = torch.stack([levels[torch.randperm(C, generator=g)] for _ in range(V)])
         E[:, C], E[:, C + 1] = 3.0 * torch.rand(V, generator=g) - 1.5, 1.5
     out["embed"] = E
@@ -144,8 +144,8 @@ def random_weights(cfg: dict, seed: int, sharp: float = 2.0) -> dict:
             n, ff = f["router"]["experts"], f["expert"]["ff"]
             R = mat(n, W, 0.1)
             R[:, coded] = 0.0
-            R[:, :n] = 16.0 * torch.eye(n)
-            R[:, C], R[:, C + 1] = 2.0, -15.5
+            R[:, :n] = 14.0 * torch.eye(n)
+            R[:, C], R[:, C + 1] = 2.0, -14.0
             out[p + "mlp.router"] = R
             for e in range(n):
                 q = f"{p}mlp.e{e}."

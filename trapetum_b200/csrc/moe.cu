@@ -67,7 +67,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(MoeRouteArgs a) {
         for (; sp < a.splits; sp++) d += src[(size_t)sp * a.split_stride];
         if (a.bias != nullptr && e < a.E) d += a.bias[e];
         const float s = 1.f / (1.f + expf(-d));
-        if (e < a.E) { score[e] = a.softmax ? d : s; choice[e] = s + (a.correction ? a.correction[e] : 0.f); }
+        // without a correction and groups the choice goes by the logit itself: in its order, and large ones whose sigmoids
+        // are the same 32-bit number still differ
+        if (e < a.E) { score[e] = a.softmax ? d : s; choice[e] = a.correction ? s + a.correction[e] : a.groups > 1 ? s : d; }
         else a.gate[t] = s;
     }
     __syncwarp();
