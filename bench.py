@@ -1396,8 +1396,11 @@ def sezanex_kernels(torch, size, hbm_gbs, tokens=PREFILL_TOKENS):
                 like="experts (weight on the output)" + what if on == "input" else None)
     # ---- the product that replaces the stream
     both, win_w = rb(T, 2 * W), rb(W, 2 * W) * .02
+    act, wdn = rb(T, ff), rb(W, ff) * .02
+    rec("down product", _median_us(torch, lambda: ops.gemm_tc(act, wdn, torch.float32, partials=True), flush), 2 * (ff * W + ff * T) + 4 * T * W,
+        tensor_flops=2.0 * T * W * ff)
     rec("loop.in product", _median_us(torch, lambda: ops.gemm_tc(both, win_w, torch.float32, partials=True), flush), 2 * (2 * W * W + 2 * T * W) + 4 * T * W,
-        tensor_flops=4.0 * T * W * W, like="up product with relu2")
+        tensor_flops=4.0 * T * W * W, like="down product")
     return out
 
 

@@ -27,7 +27,7 @@ _route = plain.route
 
 @pytest.fixture(scope="module")
 def weights():
-    return {name: random_weights(cfg, 17 + ord(name)) for name, cfg in CONFIGS.items()}
+    return {name: random_weights(cfg, 23 + ord(name)) for name, cfg in CONFIGS.items()}
 
 
 @pytest.fixture(scope="module")

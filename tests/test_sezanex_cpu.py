@@ -36,7 +36,7 @@ def test_every_constant_comes_from_the_configuration():
     assert (a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window, a.rot.dims, a.rot.base) == (4, 2, 12, 8, 0.4, 33, 12, 1000.0)
     assert a.rot.scaling == {"factor": 3.0, "original": 128.0, "fast": 8.0, "slow": 1.0}
     m = cfg.layers[2].mixer
-    assert (m.heads, m.vdim, m.state, m.groups, m.conv, m.norm_groups) == (4, 6, 16, 4, 5, 3)
+    assert (m.heads, m.vdim, m.state, m.groups, m.conv, m.norm_groups) == (4, 15, 16, 4, 5, 3)
     assert cfg.layers[2].mlp is None and cfg.layers[1].mlp.ff == 40
     assert (cfg.layers[0].mlp.experts, cfg.layers[0].mlp.top, cfg.layers[0].mlp.ff) == (5, 2, 24)
     bare = SezanexConfig.from_dict(CONFIGS["C"])
@@ -67,7 +67,7 @@ def test_a_repeated_span_is_a_schedule_in_which_every_call_owns_its_cache():
     (lambda c: c["layers"][3]["mixer"].__setitem__("kv_heads", 3), "kv_heads"),
     (lambda c: c["layers"][1]["mixer"].pop("state"), "layers[1].mixer.state"),
     (lambda c: c["layers"][2]["mixer"].__setitem__("groups", 3), "groups=3"),
-    (lambda c: c["layers"][2]["mixer"].__setitem__("norm_groups", 5), "norm_groups=5"),
+    (lambda c: c["layers"][2]["mixer"].__setitem__("norm_groups", 7), "norm_groups=7"),
     (lambda c: c["layers"][0]["mlp"].__setitem__("kind", "glu"), "known kinds: dense, moe"),
     (lambda c: c["layers"][0]["mlp"]["router"].__setitem__("top", 6), "top=6 of experts=5"),
     (lambda c: c["layers"][1]["mlp"].pop("ff"), "layers[1].mlp.ff"),
@@ -158,7 +158,7 @@ def test_the_test_models_route_without_close_calls(name):
     """What the comparisons in 16 bits rest on: no winner changes for a rounding; and the scores are neither all one nor all
     zero, so that a missing or doubled weight shows."""
     cfg = CONFIGS[name]
-    for seed in (17 + ord(name), 3):
+    for seed in (23 + ord(name), 3):
         w = doubles(random_weights(cfg, seed))
         ids = prompts(cfg["vocab"], [200], seed=seed)[0]
         assert plain.routing_margin(cfg, w, ids) > 0.3

@@ -14,7 +14,7 @@
 //             from 1: x is read from `a` instead of h and h is not touched (a norm on its own).
 //
 // No number waits for any other, so nothing is shared: a thread owns four columns (one where rows are not whole 16-byte
-// pieces) of up to four rows, keeps the columns' weights in registers and has all of its rows on their way at once.
+// pieces) of one or two rows, keeps the columns' weights in registers and has all of its rows on their way at once.
 // Everything is 32-bit; only `out` is rounded.
 #include "common.cuh"
 
@@ -140,16 +140,17 @@ extern "C" int tb_dyt(const DytArgs* args, int a_dtype, int out_dtype, cudaStrea
         && (a.give == 0 || ((uintptr_t)a.out % (4 * eo) == 0 && a.out_stride % 4 == 0))
         && (uintptr_t)a.wa % 16 == 0 && (uintptr_t)a.ba % 16 == 0 && (uintptr_t)a.wb % 16 == 0 && (uintptr_t)a.bb % 16 == 0;
     const int cols = vec ? a.width / 4 : a.width;
-    // few rows: one a thread, so that the launch spreads over the device; many: four a thread
+    // few rows: one a thread, so that the launch spreads over the device; many: two a thread (measured at 2,048 rows of
+    // 1,024 to 4,096 numbers: 13, 18 and 30 us, with four rows and 192 threads 15, 22 and 36)
     const bool many = a.rows >= 256;
-    const int threads = many ? 192 : 64;
-    const int rpt = many ? 4 : 1;
+    const int threads = many ? 128 : 64;
+    const int rpt = many ? 2 : 1;
     const dim3 grid((a.rows + rpt - 1) / rpt, (cols + threads - 1) / threads);
     if (grid.y > 65535) return tb_refuse("dyt: rows of %d numbers are too wide", a.width);
 #define GO(TA, TO) do { \
-        if (vec && many) tb_launch(dyt_kernel<TA, TO, 4, 4>, grid, dim3(threads), 0, stream, a); \
+        if (vec && many) tb_launch(dyt_kernel<TA, TO, 4, 2>, grid, dim3(threads), 0, stream, a); \
         else if (vec) tb_launch(dyt_kernel<TA, TO, 4, 1>, grid, dim3(threads), 0, stream, a); \
-        else if (many) tb_launch(dyt_kernel<TA, TO, 1, 4>, grid, dim3(threads), 0, stream, a); \
+        else if (many) tb_launch(dyt_kernel<TA, TO, 1, 2>, grid, dim3(threads), 0, stream, a); \
         else tb_launch(dyt_kernel<TA, TO, 1, 1>, grid, dim3(threads), 0, stream, a); } while (0)
     TB_DISPATCH_1(a_dtype, TA, TB_DISPATCH_1(out_dtype, TO, GO(TA, TO)));
 #undef GO
