@@ -269,7 +269,7 @@ def test_the_exact_gelu_in_its_kernel_and_in_the_products_epilogue(dtype):
             near(ops.gemm_tc(dev(x), dev(w), torch.bfloat16, unary_act="gelu"), want, "bfloat16", f"product of {T} x {N} x {K}", rel16=4e-3)
 
 
-@pytest.mark.parametrize("E, top", [(5, 2), (4, 4), (12, 1), (1, 1), (64, 6), (40, 33)])
+@pytest.mark.parametrize("E, top", [(5, 2), (4, 4), (11, 1), (1, 1), (64, 6), (40, 33)])
 def test_scores_as_weights(E, top):
     from trapetum_b200.csrc import ops
     g = torch.Generator().manual_seed(E * top)
